@@ -1,17 +1,70 @@
 #!/usr/bin/env bash
-# Builds lib/libmllm_b200.so (CUDA kernels + C ABI) for sm_100a, in tree.
+# Builds the sm_100a libraries (CUDA kernels + C ABI) in tree, one object per source, in parallel:
+#   lib/libmllm_b200.so     quantized linears, the quantized decoder, tensor parallelism   (include/mllmb200.h)
+#   lib/libmllm_b200_lm.so  bf16 language-model engine                                     (include/mllmb200_lm.h)
+# Usage: build.sh [all|core|lm].  Objects whose sources have not changed are kept.
 set -euo pipefail
 HERE="$(cd "$(dirname "${BASH_SOURCE[0]}")" && pwd)"
 NVCC="${NVCC:-/usr/local/cuda/bin/nvcc}"
+[ -x "$NVCC" ] || NVCC=nvcc
+WHAT="${1:-all}"
 OUT="$HERE/lib"
-mkdir -p "$OUT"
-SRC=("$HERE"/csrc/host_pack.cpp "$HERE"/csrc/c_api.cu "$HERE"/csrc/repack.cu "$HERE"/csrc/act_quant.cu
-     "$HERE"/csrc/gemv.cu "$HERE"/csrc/gemv_stream.cu "$HERE"/csrc/gemm_stream.cu "$HERE"/csrc/gemm_simt.cu "$HERE"/csrc/gemm_tc.cu "$HERE"/csrc/gemm_tcf16.cu
-     "$HERE"/csrc/decoder_kernels.cu "$HERE"/csrc/decoder_attn.cu "$HERE"/csrc/decoder.cu "$HERE"/csrc/decoder_batch.cu "$HERE"/csrc/decoder_persistent.cu "$HERE"/csrc/conv3d.cu
-     "$HERE"/csrc/host_pack_a16.cpp "$HERE"/csrc/w4a16.cu "$HERE"/csrc/c_api_a16.cu "$HERE"/csrc/tp.cu)
-EXTRA=()
-[ -f "$HERE/csrc/no_alloc.cu" ] && SRC+=("$HERE/csrc/no_alloc.cu")
-"$NVCC" -std=c++17 -O3 -gencode arch=compute_100a,code=sm_100a -lineinfo -rdc=true \
-  -Xcompiler -fPIC,-fvisibility=hidden,-O3 ${PTXAS_V:+-Xptxas -v} \
-  -shared -o "$OUT/libmllm_b200.so" "${SRC[@]}" "${EXTRA[@]}" -ldl
-echo "built $OUT/libmllm_b200.so"
+OBJ="$HERE/build"
+mkdir -p "$OUT" "$OBJ"
+CORE=(host_pack.cpp c_api.cu device_status.cu repack.cu act_quant.cu gemv.cu gemv_stream.cu gemm_stream.cu gemm_simt.cu gemm_tc.cu
+      gemm_tcf16.cu decoder_kernels.cu decoder_attn.cu decoder_sample.cu decoder.cu decoder_batch.cu decoder_persistent.cu conv3d.cu
+      host_pack_a16.cpp w4a16.cu c_api_a16.cu tp.cu)
+[ -f "$HERE/csrc/no_alloc.cu" ] && CORE+=(no_alloc.cu)
+LM=(lm/lm_engine.cu lm/lm_linear.cu lm/lm_norm.cu lm/lm_attn.cu lm/lm_retention.cu device_status.cu decoder_sample.cu)
+FLAGS=(-std=c++17 -O3 -gencode arch=compute_100a,code=sm_100a -lineinfo -rdc=true -Xcompiler -fPIC,-fvisibility=hidden,-O3)
+[ -n "${PTXAS_V:-}" ] && FLAGS+=(-Xptxas -v)
+
+# what an object depends on: every header, its own source, the flags
+HEADERS="$(cat "$HERE"/csrc/*.h "$HERE"/csrc/*.cuh "$HERE"/csrc/*.inc "$HERE"/csrc/lm/*.h "$HERE"/../include/*.h | sha256sum)"
+compile() {
+  local src="$1" obj stamp
+  obj="$OBJ/$(echo "$src" | tr '/.' '__').o"
+  stamp="$(echo "$HEADERS ${FLAGS[*]} $(sha256sum <"$HERE/csrc/$src")" | sha256sum)"
+  [ -f "$obj" ] && [ "$(cat "$obj.stamp" 2>/dev/null)" = "$stamp" ] && return 0
+  "$NVCC" "${FLAGS[@]}" -c "$HERE/csrc/$src" -o "$obj.$$.o"
+  mv "$obj.$$.o" "$obj"
+  echo "$stamp" >"$obj.stamp"
+}
+link() {
+  local lib="$1"
+  shift
+  local objs=()
+  for s in "$@"; do objs+=("$OBJ/$(echo "$s" | tr '/.' '__').o"); done
+  "$NVCC" -gencode arch=compute_100a,code=sm_100a -shared -o "$OUT/$lib.$$" "${objs[@]}" -ldl
+  mv "$OUT/$lib.$$" "$OUT/$lib"
+  echo "built $OUT/$lib"
+}
+
+case "$WHAT" in
+  all) SRC=("${CORE[@]}" "${LM[@]}") ;;
+  core) SRC=("${CORE[@]}") ;;
+  lm) SRC=("${LM[@]}") ;;
+  *) echo "usage: build.sh [all|core|lm]" >&2; exit 2 ;;
+esac
+# One build at a time; nothing to do when the libraries are those of these sources.
+exec 9>"$OBJ/.lock"
+flock 9
+STAMP="$(cd "$HERE/csrc" && echo "$HEADERS ${FLAGS[*]} $(sha256sum "${SRC[@]}")" | sha256sum)"
+if [ "$(cat "$OUT/.$WHAT.stamp" 2>/dev/null)" = "$STAMP" ] && { [ "$WHAT" = lm ] || [ -f "$OUT/libmllm_b200.so" ]; } &&
+   { [ "$WHAT" = core ] || [ -f "$OUT/libmllm_b200_lm.so" ]; }; then
+  exit 0
+fi
+JOBS="$(nproc)"
+rm -f "$OBJ/.failed"
+declare -A started=()
+for s in "${SRC[@]}"; do
+  [ -n "${started[$s]:-}" ] && continue
+  started[$s]=1
+  while [ "$(jobs -rp | wc -l)" -ge "$JOBS" ]; do wait -n || true; done
+  { compile "$s" || touch "$OBJ/.failed"; } 9>&- &
+done
+wait
+[ ! -e "$OBJ/.failed" ] || { echo "build.sh: a source did not compile" >&2; exit 1; }
+[ "$WHAT" = lm ] || link libmllm_b200.so "${CORE[@]}"
+[ "$WHAT" = core ] || link libmllm_b200_lm.so "${LM[@]}"
+echo "$STAMP" >"$OUT/.$WHAT.stamp"

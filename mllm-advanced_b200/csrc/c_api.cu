@@ -54,6 +54,8 @@ cudaError_t launch_w4a32_gemm_stream(const uint8_t*, const float2*, int, int, in
                                      const int*, const int*, int, cudaStream_t);
 constexpr int kStreamGemmMinM = 5, kStreamGemmMaxM = 64;  // batch sizes the streaming tensor-core GEMM takes by default
 
+cudaError_t read_device_status(cudaStream_t, int* status);
+
 static thread_local int t_last_cuda_error = 0;
 static int cuda_fail(cudaError_t e) {
   t_last_cuda_error = (int)e;
@@ -395,18 +397,9 @@ int mllmb200_selftest_wait_timeout(long long limit_ticks, int* gave_up_dev, void
 }
 
 int mllmb200_check_device_status(void* stream) {
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  cudaError_t e = cudaStreamSynchronize(st);
-  if (e != cudaSuccess) return cuda_fail(e);
-  unsigned int word = 0;
-  if ((e = cudaMemcpyFromSymbol(&word, g_device_status, sizeof(word))) != cudaSuccess) return cuda_fail(e);
-  if (word != 0) {
-    const unsigned int zero = 0;
-    if ((e = cudaMemcpyToSymbol(g_device_status, &zero, sizeof(zero))) != cudaSuccess) return cuda_fail(e);
-  }
-  if (word & kDevStatusTimeout) return MLLMB200_TIMEOUT;
-  if (word & kDevStatusBadHeader) return MLLMB200_BAD_BLOB;
-  return MLLMB200_OK;
+  int status = MLLMB200_OK;
+  const cudaError_t e = read_device_status(static_cast<cudaStream_t>(stream), &status);
+  return e != cudaSuccess ? cuda_fail(e) : status;
 }
 
 }  // extern "C"

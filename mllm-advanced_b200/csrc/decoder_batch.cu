@@ -41,6 +41,7 @@ __global__ void add_rmsnorm_quant_kernel(const float*, const float*, const float
                                          float2*, int);
 __global__ void silu_mul_quant_kernel(const float*, const float*, int, float*, uint8_t*, float2*, int);
 __global__ void embedding_kernel(const int*, const float*, int, float*);
+__global__ void sample_advance_batched_kernel(const float2*, int, int*, int*, int*, int, const int*, int*);
 
 // Decode-step attention for a batch: grid (splits, kv_heads, sequences), 256 threads; the work of a CTA is
 // attn_partial_body on the sequence's own cache and position.
@@ -436,38 +437,6 @@ __global__ void __launch_bounds__(kLmThreads, 1) lm_head_f16_batched_kernel(cons
   }
 }
 
-// Greedy sampling and bookkeeping of a step for every sequence (one warp each): sample_advance_kernel per row.
-__global__ void sample_advance_batched_kernel(const float2* __restrict__ best, int count, int* __restrict__ pos,
-                                              int* __restrict__ token, int* __restrict__ history, int max_hist) {
-  const int seq = blockIdx.x;
-  best += (size_t)seq * count;
-  float bv = -3.402823466e+38f;
-  int bi = 0x7fffffff;
-  for (int i = threadIdx.x; i < count; i += 32) {
-    const float2 c = best[i];
-    const int ci = __float_as_int(c.y);
-    if (c.x > bv || (c.x == bv && ci < bi)) {
-      bv = c.x;
-      bi = ci;
-    }
-  }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-    if (ov > bv || (ov == bv && oi < bi)) {
-      bv = ov;
-      bi = oi;
-    }
-  }
-  if (threadIdx.x == 0) {
-    const int p = pos[seq];
-    token[seq] = bi;
-    if (p < max_hist) history[(size_t)seq * max_hist + p] = bi;
-    pos[seq] = p + 1;
-  }
-}
-
 namespace {
 
 constexpr int kLmCtas = 148;  // vocabulary CTAs of the batched lm_head (x ceil(B / 32) activation tiles)
@@ -568,7 +537,7 @@ int enqueue_batched_step(BatchDecoder* b) {
     lm_head_f16_batched_kernel<<<grid, kLmThreads, lm_smem_bytes(H), s>>>(b->xn, B, d->lm_head, H, c.vocab,
                                                                                       b->logits, b->best);
   }
-  sample_advance_batched_kernel<<<B, 32, 0, s>>>(b->best, kLmCtas, b->pos, b->token, b->history, c.max_ctx);
+  sample_advance_batched_kernel<<<B, 32, 0, s>>>(b->best, kLmCtas, b->pos, b->token, b->history, c.max_ctx, nullptr, nullptr);
   BD_CHECK(cudaGetLastError());
   return MLLMB200_OK;
 }

@@ -1,0 +1,222 @@
+// Row operators of the language-model engine: embedding, sandwich norm with residual and causal input convolution,
+// the bookkeeping of a decode step, and the argmax candidates of greedy sampling.
+#include <algorithm>
+
+#include "../device_common.cuh"
+#include "lm_state.h"
+
+namespace mllmb200 {
+namespace lm {
+namespace {
+
+constexpr int kNormThreads = 256;
+
+__device__ __forceinline__ float block_sum(float v, float* scratch) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();
+  if (lane == 0) scratch[warp] = v;
+  __syncthreads();
+  float t = lane < (int)(blockDim.x >> 5) ? scratch[lane] : 0.0f;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+  return t;
+}
+
+__device__ __forceinline__ float4 fma4(float s, const float4& a, const float4& b) {
+  return make_float4(fmaf(s, a.x, b.x), fmaf(s, a.y, b.y), fmaf(s, a.z, b.z), fmaf(s, a.w, b.w));
+}
+__device__ __forceinline__ float dot4(const float4& a) { return a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w; }
+
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+// x' = x + rms_unit(delta) * g_post;  h = rms_unit(x') * g_pre;  out = h + conv(h).
+// The gains are one number per norm.  A CTA walks `rows_per_cta` rows in order and keeps the last taps rows of h in
+// shared memory; the taps - 1 rows in front of its first one are recomputed (x_in is not overwritten: x_out is another
+// buffer), or come from the sequence's tail when they belong to an earlier step.  A thread owns the same columns of
+// every row, so the ring needs no synchronization.  The CTA with a sequence's last row writes the new tail, into the
+// other of the sequence's two tail buffers (another CTA may still read the old one).
+template <class T, int NV>
+__global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
+  extern __shared__ __align__(16) float ring[];  // [taps][ldx]
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int tid = threadIdx.x, nv = a.ldx >> 2;
+  const float g_pre = *a.g_pre, g_post = a.delta ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
+  const int r_begin = blockIdx.x * a.rows_per_cta, r_end = min(r_begin + a.rows_per_cta, a.rows);
+  int t0 = r_begin;
+  if (a.taps > 1) t0 = max(r_begin - (a.taps - 1), a.entries[a.row_entry[r_begin]].row0);
+  for (int t = t0; t < r_end; ++t) {
+    const int src = a.gather ? a.gather[t] : t;
+    const float* xr = a.x_in + (size_t)src * a.ldx;
+    float4 x[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = tid + i * kNormThreads;
+      x[i] = c < nv ? reinterpret_cast<const float4*>(xr)[c] : make_float4(0, 0, 0, 0);
+    }
+    if (a.delta) {
+      float4 d[NV];
+      float ss = 0.0f;
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = tid + i * kNormThreads;
+        d[i] = make_float4(0, 0, 0, 0);
+        if (c < nv) {
+          const float* dr = a.delta + (size_t)src * a.ldx + c * 4;
+          d[i] = *reinterpret_cast<const float4*>(dr);
+          for (int p = 1; p < a.planes; ++p) d[i] = fma4(1.0f, *reinterpret_cast<const float4*>(dr + p * a.plane), d[i]);
+          ss += dot4(d[i]);
+        }
+      }
+      const float r = g_post / sqrtf(block_sum(ss, scratch) * inv_w + a.eps);
+#pragma unroll
+      for (int i = 0; i < NV; ++i) x[i] = fma4(r, d[i], x[i]);
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += dot4(x[i]);
+    const float r = g_pre / sqrtf(block_sum(ss, scratch) * inv_w + a.eps);
+    const bool own = t >= r_begin;
+    if (own && a.x_out) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = tid + i * kNormThreads;
+        if (c < nv) store4(a.x_out + (size_t)t * a.ldx + c * 4, x[i]);
+      }
+    }
+    T* out = static_cast<T*>(a.out) + (size_t)t * a.ldx;
+    if (a.taps == 0) {
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = tid + i * kNormThreads;
+        if (c < nv) store4(out + c * 4, fma4(r, x[i], make_float4(0, 0, 0, 0)));
+      }
+      continue;
+    }
+    const Entry e = a.entries[a.row_entry[t]];
+    const int off = t - e.row0, keep = a.taps - 1;
+    const float* old_tail = a.tail + ((size_t)e.slot * 2 + e.tail) * keep * a.ldx;
+    float* new_tail = a.tail + ((size_t)e.slot * 2 + (e.tail ^ 1)) * keep * a.ldx;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = tid + i * kNormThreads;
+      if (c >= nv) continue;
+      const float4 h = fma4(r, x[i], make_float4(0, 0, 0, 0));
+      store4(ring + (size_t)(t % a.taps) * a.ldx + c * 4, h);
+      if (!own) continue;
+      float4 y = h;
+      for (int s = 0; s < a.taps; ++s) {
+        float4 hs;
+        if (s <= off) hs = *reinterpret_cast<const float4*>(ring + (size_t)((t - s) % a.taps) * a.ldx + c * 4);
+        else if (s <= e.pos0 + off) hs = *reinterpret_cast<const float4*>(old_tail + (size_t)(keep - (s - off)) * a.ldx + c * 4);
+        else break;  // before the start of the sequence
+        const float4 w = *reinterpret_cast<const float4*>(a.conv_w + (size_t)(keep - s) * a.ldx + c * 4);
+        y = make_float4(fmaf(w.x, hs.x, y.x), fmaf(w.y, hs.y, y.y), fmaf(w.z, hs.z, y.z), fmaf(w.w, hs.w, y.w));
+      }
+      store4(out + c * 4, y);
+      const int at = keep - (e.count - off);
+      if (at >= 0) store4(new_tail + (size_t)at * a.ldx + c * 4, h);
+      if (off == e.count - 1)  // a short step: older rows move down
+        for (int j = 0; j + e.count < keep; ++j)
+          store4(new_tail + (size_t)j * a.ldx + c * 4, *reinterpret_cast<const float4*>(old_tail + (size_t)(j + e.count) * a.ldx + c * 4));
+    }
+  }
+}
+
+template <class T, int NV>
+cudaError_t launch_norm_nv(cudaStream_t s, const NormArgs& a) {
+  const size_t smem = (size_t)a.taps * a.ldx * sizeof(float);
+  if (smem > 48 * 1024) {
+    const cudaError_t r = cudaFuncSetAttribute(lm_norm_kernel<T, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (r != cudaSuccess) return r;
+  }
+  return launch_pdl(lm_norm_kernel<T, NV>, dim3((a.rows + a.rows_per_cta - 1) / a.rows_per_cta), dim3(kNormThreads), smem, s, a);
+}
+template <class T>
+cudaError_t launch_norm_t(cudaStream_t s, const NormArgs& a) {
+  const int per = (a.ldx / 4 + kNormThreads - 1) / kNormThreads;
+  if (per <= 1) return launch_norm_nv<T, 1>(s, a);
+  if (per <= 2) return launch_norm_nv<T, 2>(s, a);
+  if (per <= 4) return launch_norm_nv<T, 4>(s, a);
+  if (per <= 8) return launch_norm_nv<T, 8>(s, a);
+  return cudaErrorInvalidValue;
+}
+
+__global__ void lm_embed_kernel(const int* __restrict__ tokens, const __nv_bfloat16* __restrict__ table, int width, int ldx,
+                                float* __restrict__ x) {
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const __nv_bfloat16* src = table + (size_t)tokens[blockIdx.x] * width;
+  for (int k = threadIdx.x; k < ldx; k += blockDim.x)
+    x[(size_t)blockIdx.x * ldx + k] = k < width ? __bfloat162float(src[k]) : 0.0f;
+}
+
+// Rows of a decode step: one token per slot, from the slots' own state.
+__global__ void lm_decode_prep_kernel(int n, const int* __restrict__ slots, const int* __restrict__ pos, const int* __restrict__ token,
+                                      const int* __restrict__ flip, int2* __restrict__ row_sp, int* __restrict__ row_token,
+                                      Entry* __restrict__ entries, int* __restrict__ row_entry) {
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int b = blockIdx.x * blockDim.x + threadIdx.x;
+  if (b >= n) return;
+  const int slot = slots[b], p = pos[slot];
+  row_sp[b] = make_int2(slot, p);
+  row_token[b] = token[slot];
+  entries[b] = Entry{slot, p, b, 1, flip[slot]};
+  row_entry[b] = b;
+}
+
+// The largest logit of each of gridDim.x ranges of the vocabulary (lowest index on ties); gridDim.y rows.
+__global__ void __launch_bounds__(256) lm_argmax_kernel(const float* __restrict__ logits, int vocab, float2* __restrict__ best) {
+  __shared__ float sv[8];
+  __shared__ int si[8];
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const float* row = logits + (size_t)blockIdx.y * vocab;
+  float bv = -3.402823466e+38f;
+  int bi = 0x7fffffff;
+  for (int i = blockIdx.x * 256 + threadIdx.x; i < vocab; i += gridDim.x * 256)
+    if (row[i] > bv) bv = row[i], bi = i;
+  auto merge = [&](float ov, int oi) {
+    if (ov > bv || (ov == bv && oi < bi)) bv = ov, bi = oi;
+  };
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+    merge(ov, oi);
+  }
+  if ((threadIdx.x & 31) == 0) sv[threadIdx.x >> 5] = bv, si[threadIdx.x >> 5] = bi;
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    for (int i = 1; i < 8; ++i) merge(sv[i], si[i]);
+    best[(size_t)blockIdx.y * gridDim.x + blockIdx.x] = make_float2(bv, __int_as_float(bi));
+  }
+}
+
+}  // namespace
+
+cudaError_t launch_norm(cudaStream_t s, bool f32, const NormArgs& a) {
+  return f32 ? launch_norm_t<float>(s, a) : launch_norm_t<__nv_bfloat16>(s, a);
+}
+cudaError_t launch_embed(cudaStream_t s, const int* tokens, const __nv_bfloat16* table, int width, int ldx, int rows, float* x) {
+  return launch_pdl(lm_embed_kernel, dim3(rows), dim3(256), 0, s, tokens, table, width, ldx, x);
+}
+cudaError_t launch_decode_prep(cudaStream_t s, int n, const int* slots, const int* pos, const int* token, const int* flip,
+                               int2* row_sp, int* row_token, Entry* entries, int* row_entry) {
+  return launch_pdl(lm_decode_prep_kernel, dim3((n + 127) / 128), dim3(128), 0, s, n, slots, pos, token, flip, row_sp, row_token,
+                    entries, row_entry);
+}
+cudaError_t launch_argmax(cudaStream_t s, const float* logits, int rows, int vocab, int blocks, float2* best) {
+  return launch_pdl(lm_argmax_kernel, dim3(blocks, rows), dim3(256), 0, s, logits, vocab, best);
+}
+
+}  // namespace lm
+}  // namespace mllmb200

@@ -1,0 +1,392 @@
+// Retention: linear attention with a fixed decay per head, S_t = decay S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, each head's
+// o over its root mean square, times silu of a gate.  q and k are rotated (half-split layout, first rot_dims
+// coordinates) and k is multiplied by dim^-1/2.  Everything after the projections is fp32: the rotated q and k, the
+// states, the decays (powers tabulated in double precision and rounded once) and all products.
+//   * one token per sequence: lm_ret_decode_kernel updates the state in place.
+//   * prompts and portions: chunks of kChunk tokens, cut from the portion's own start.  lm_ret_rotate_kernel rotates in
+//     place, lm_ret_chunk_kernel forms every chunk's own contribution to the state, lm_ret_scan_kernel chains them
+//     (leaving the state in front of every chunk), lm_ret_output_kernel combines the part inside the chunk with the
+//     state in front of it, and applies norm and gate.
+#include <algorithm>
+
+#include "../device_common.cuh"
+#include "lm_state.h"
+
+namespace mllmb200 {
+namespace lm {
+namespace {
+
+constexpr int kThreads = 256, kPad = kChunk + 4, kStateRows = 16;
+
+template <class T>
+__device__ __forceinline__ T from_f32(float v);
+template <>
+__device__ __forceinline__ float from_f32<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+
+// angles in double precision, one rounding of cos and sin
+__global__ void lm_rope_table_kernel(float* cos_t, float* sin_t, int max_pos, int half, double base) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= max_pos * half) return;
+  const int p = i / half, d = i - p * half;
+  const double a = (double)p * pow(base, -(double)d / (double)half);
+  double s, c;
+  sincos(a, &s, &c);
+  cos_t[i] = (float)c;
+  sin_t[i] = (float)s;
+}
+
+// coordinate d of a rotated head at position pos; x points at the head
+__device__ __forceinline__ float rotated(const float* x, int d, int rot_dims, const float* cos_r, const float* sin_r) {
+  if (d >= rot_dims) return x[d];
+  const int half = rot_dims >> 1;
+  const int i = d < half ? d : d - half;
+  const float u = x[i], v = x[i + half], c = cos_r[i], s = sin_r[i];
+  return d < half ? u * c - v * s : v * c + u * s;
+}
+
+template <class T>
+__global__ void __launch_bounds__(kThreads) lm_ret_decode_kernel(RetentionArgs a) {
+  extern __shared__ __align__(16) float dec_smem[];
+  __shared__ float wsum[kThreads / 32];
+  float *sq = dec_smem, *sk = sq + a.dimp, *sv = sk + a.dimp, *red = sv + a.vdimp;
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int h = blockIdx.x, row = blockIdx.y, tid = threadIdx.x;
+  const int2 sp = a.row_sp[row];
+  const float* qr = a.qkvg + (size_t)row * a.ld + h * a.dimp;
+  const float* kr = qr + a.heads * a.dimp;
+  const float* vr = a.qkvg + (size_t)row * a.ld + 2 * a.heads * a.dimp + h * a.vdimp;
+  const float* gr = vr + a.heads * a.vdimp;
+  const int half = a.rot_dims >> 1;
+  const float *cr = a.cos_t + (size_t)sp.y * half, *sr = a.sin_t + (size_t)sp.y * half;
+  const float decay = a.decay[h * (kChunk + 1) + 1], kscale = 1.0f / sqrtf((float)a.dim);
+  const int vl_n = a.vdimp >> 2, rg_n = kThreads / vl_n, vl = tid % vl_n, rg = tid / vl_n;
+  float* st = a.state + ((size_t)sp.x * a.heads + h) * a.dimp * a.vdimp + vl * 4;
+  const bool fresh = sp.y == 0;
+  for (int d = tid; d < a.dimp; d += kThreads) {
+    sq[d] = rotated(qr, d, a.rot_dims, cr, sr);
+    sk[d] = rotated(kr, d, a.rot_dims, cr, sr) * kscale;
+  }
+  for (int d = tid; d < a.vdimp; d += kThreads) sv[d] = vr[d];
+  __syncthreads();
+  if (rg < rg_n) {
+    const float4 v = *reinterpret_cast<const float4*>(sv + vl * 4);
+    float4 o = make_float4(0, 0, 0, 0);
+    constexpr int U = 8;
+    for (int r0 = rg; r0 < a.dim; r0 += U * rg_n) {
+      float4 s[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int r = r0 + u * rg_n;
+        s[u] = !fresh && r < a.dim ? *reinterpret_cast<const float4*>(st + (size_t)r * a.vdimp) : make_float4(0, 0, 0, 0);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int r = r0 + u * rg_n;
+        if (r >= a.dim) break;
+        const float k = sk[r], q = sq[r];
+        s[u] = make_float4(fmaf(decay, s[u].x, k * v.x), fmaf(decay, s[u].y, k * v.y), fmaf(decay, s[u].z, k * v.z),
+                           fmaf(decay, s[u].w, k * v.w));
+        *reinterpret_cast<float4*>(st + (size_t)r * a.vdimp) = s[u];
+        o = make_float4(fmaf(q, s[u].x, o.x), fmaf(q, s[u].y, o.y), fmaf(q, s[u].z, o.z), fmaf(q, s[u].w, o.w));
+      }
+    }
+    *reinterpret_cast<float4*>(red + (size_t)rg * a.vdimp + vl * 4) = o;
+  }
+  __syncthreads();
+  float o = 0.0f;
+  if (tid < a.vdimp)
+    for (int g = 0; g < rg_n; ++g) o += red[(size_t)g * a.vdimp + tid];
+  float ss = o * o;
+#pragma unroll
+  for (int i = 16; i > 0; i >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, i);
+  if ((tid & 31) == 0) wsum[tid >> 5] = ss;
+  __syncthreads();
+  ss = 0.0f;
+  for (int i = 0; i < kThreads / 32; ++i) ss += wsum[i];
+  if (tid < a.vdimp)
+    static_cast<T*>(a.out)[(size_t)row * a.ldo + h * a.vdimp + tid] =
+        from_f32<T>(o / sqrtf(ss / (float)a.vdim + a.eps) * silu(gr[tid]));
+}
+
+// grid rows: rotates q and k in place and scales k
+__global__ void __launch_bounds__(kThreads) lm_ret_rotate_kernel(RetentionArgs a) {
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int row = blockIdx.x, pos = a.row_sp[row].y, half = a.rot_dims >> 1, rest = a.dim - a.rot_dims;
+  const float *cr = a.cos_t + (size_t)pos * half, *sr = a.sin_t + (size_t)pos * half;
+  const float kscale = 1.0f / sqrtf((float)a.dim);
+  float* base = a.qkvg + (size_t)row * a.ld;
+  for (int i = threadIdx.x; i < 2 * a.heads * half; i += kThreads) {
+    const int h = i / half, d = i - h * half;
+    float* x = base + (size_t)h * a.dimp;
+    const float f = h < a.heads ? 1.0f : kscale;
+    const float u = x[d], v = x[d + half], c = cr[d], s = sr[d];
+    x[d] = (u * c - v * s) * f;
+    x[d + half] = (v * c + u * s) * f;
+  }
+  for (int i = threadIdx.x; i < a.heads * rest; i += kThreads) {
+    const int h = i / rest;
+    base[(size_t)(a.heads + h) * a.dimp + a.rot_dims + (i - h * rest)] *= kscale;
+  }
+}
+
+// acc[r][c] += A[k][4 ty + r] * B[k][4 tx + 64 i + c], both from shared memory
+template <int NC>
+__device__ __forceinline__ void tile_fma(float (&acc)[4][4 * NC], const float* A, int lda, const float* B, int ldb, int n, int ty, int tx,
+                                         int cols) {
+#pragma unroll 4
+  for (int k = 0; k < n; ++k) {
+    const float4 av = *reinterpret_cast<const float4*>(A + (size_t)k * lda + ty * 4);
+    const float ar[4] = {av.x, av.y, av.z, av.w};
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = tx * 4 + i * 64;
+      if (c < cols) {
+        const float4 b = *reinterpret_cast<const float4*>(B + (size_t)k * ldb + c);
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          acc[r][4 * i] = fmaf(ar[r], b.x, acc[r][4 * i]);
+          acc[r][4 * i + 1] = fmaf(ar[r], b.y, acc[r][4 * i + 1]);
+          acc[r][4 * i + 2] = fmaf(ar[r], b.z, acc[r][4 * i + 2]);
+          acc[r][4 * i + 3] = fmaf(ar[r], b.w, acc[r][4 * i + 3]);
+        }
+      }
+    }
+  }
+}
+
+struct ChunkPos {
+  int row0, len;
+};
+__device__ __forceinline__ ChunkPos chunk_pos(const RetentionArgs& a, int chunk) {
+  const int2 c = a.chunks[chunk];
+  const Entry e = a.entries[c.x];
+  return {e.row0 + c.y, min(kChunk, e.count - c.y)};
+}
+
+// grid (chunks, heads, blocks of 64 state rows): sum over the chunk of decay^(len-1-j) k_j v_j^T
+template <int NC>
+__global__ void __launch_bounds__(kThreads) lm_ret_chunk_kernel(RetentionArgs a) {
+  extern __shared__ __align__(16) float ck_smem[];
+  float *sK = ck_smem, *sV = sK + kChunk * 64;  // [kChunk][64], [kChunk][vdimp]
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int chunk = blockIdx.x, h = blockIdx.y, d0 = blockIdx.z * 64, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const ChunkPos p = chunk_pos(a, chunk);
+  const float* pw = a.decay + h * (kChunk + 1);
+  const float* kb = a.qkvg + (size_t)p.row0 * a.ld + (a.heads + h) * a.dimp;
+  const float* vb = a.qkvg + (size_t)p.row0 * a.ld + 2 * a.heads * a.dimp + h * a.vdimp;
+  const int nd = min(64, a.dimp - d0), v4 = a.vdimp / 4;
+  for (int i = tid; i < p.len * 16; i += kThreads) {
+    const int j = i >> 4, c = (i & 15) * 4;
+    float4 k = make_float4(0, 0, 0, 0);
+    if (c < nd) k = *reinterpret_cast<const float4*>(kb + (size_t)j * a.ld + d0 + c);
+    const float f = pw[p.len - 1 - j];
+    *reinterpret_cast<float4*>(sK + j * 64 + c) = make_float4(k.x * f, k.y * f, k.z * f, k.w * f);
+  }
+  for (int i = tid; i < p.len * v4; i += kThreads) {
+    const int j = i / v4, c = (i - j * v4) * 4;
+    *reinterpret_cast<float4*>(sV + j * a.vdimp + c) = *reinterpret_cast<const float4*>(vb + (size_t)j * a.ld + c);
+  }
+  __syncthreads();
+  float acc[4][4 * NC] = {};
+  tile_fma<NC>(acc, sK, 64, sV, a.vdimp, p.len, ty, tx, a.vdimp);
+  float* dst = a.chunk_state + ((size_t)chunk * a.heads + h) * a.dimp * a.vdimp;
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    const int d = d0 + ty * 4 + r;
+    if (d >= a.dimp) break;
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = tx * 4 + i * 64;
+      if (c < a.vdimp)
+        *reinterpret_cast<float4*>(dst + (size_t)d * a.vdimp + c) = make_float4(acc[r][4 * i], acc[r][4 * i + 1], acc[r][4 * i + 2], acc[r][4 * i + 3]);
+    }
+  }
+}
+
+// grid (blocks of 256 float4 of a state, heads, entries): chunk_state becomes the state in front of each chunk
+__global__ void __launch_bounds__(kThreads) lm_ret_scan_kernel(RetentionArgs a) {
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int i = blockIdx.x * kThreads + threadIdx.x, h = blockIdx.y;
+  const size_t n4 = (size_t)a.dimp * a.vdimp / 4;
+  if (i >= (int)n4) return;
+  const Entry e = a.entries[blockIdx.z];
+  const int2 ec = a.entry_chunks[blockIdx.z];
+  float4* st = reinterpret_cast<float4*>(a.state) + ((size_t)e.slot * a.heads + h) * n4 + i;
+  float4 s = e.pos0 == 0 ? make_float4(0, 0, 0, 0) : *st;
+  float4* cs = reinterpret_cast<float4*>(a.chunk_state) + ((size_t)ec.x * a.heads + h) * n4 + i;
+  const size_t step = (size_t)a.heads * n4;
+  for (int c0 = 0; c0 < ec.y; c0 += 8) {
+    float4 u[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      if (c0 + j < ec.y) u[j] = cs[(size_t)(c0 + j) * step];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      if (c0 + j >= ec.y) break;
+      const float f = a.decay[h * (kChunk + 1) + min(kChunk, e.count - (c0 + j) * kChunk)];
+      cs[(size_t)(c0 + j) * step] = s;
+      s = make_float4(fmaf(f, s.x, u[j].x), fmaf(f, s.y, u[j].y), fmaf(f, s.z, u[j].z), fmaf(f, s.w, u[j].w));
+    }
+  }
+  *st = s;
+}
+
+size_t output_smem(const RetentionArgs& a) {
+  const size_t shared_part = std::max((size_t)a.dimp * kPad, (size_t)kChunk * kPad + (size_t)kStateRows * a.vdimp);
+  return ((size_t)a.dimp * kPad + shared_part + (size_t)kChunk * a.vdimp) * 4;
+}
+
+// grid (chunks, heads)
+template <class T, int NC>
+__global__ void __launch_bounds__(kThreads) lm_ret_output_kernel(RetentionArgs a) {
+  extern __shared__ __align__(16) float out_smem[];
+  float* sQ = out_smem;                        // [dimp][kPad]: q transposed
+  float* sV = sQ + (size_t)a.dimp * kPad;      // [kChunk][vdimp]
+  float* sK = sV + (size_t)kChunk * a.vdimp;   // [dimp][kPad]: k transposed; afterwards
+  float* sA = sK;                              //   [kChunk][kPad]: decayed scores, transposed
+  float* sS = sA + (size_t)kChunk * kPad;      //   [kStateRows][vdimp]: rows of the state
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+  const ChunkPos p = chunk_pos(a, chunk);
+  const float* pw = a.decay + h * (kChunk + 1);
+  const float* qb = a.qkvg + (size_t)p.row0 * a.ld + h * a.dimp;
+  const float* kb = qb + a.heads * a.dimp;
+  const float* vb = a.qkvg + (size_t)p.row0 * a.ld + 2 * a.heads * a.dimp + h * a.vdimp;
+  const float* gb = vb + a.heads * a.vdimp;
+  const int d4 = a.dimp / 4, v4 = a.vdimp / 4;
+  for (int i = tid; i < kChunk * d4; i += kThreads) {
+    const int j = i / d4, d = (i - j * d4) * 4;
+    float4 q = make_float4(0, 0, 0, 0), k = q;
+    if (j < p.len) {
+      q = *reinterpret_cast<const float4*>(qb + (size_t)j * a.ld + d);
+      k = *reinterpret_cast<const float4*>(kb + (size_t)j * a.ld + d);
+    }
+    sQ[d * kPad + j] = q.x, sQ[(d + 1) * kPad + j] = q.y, sQ[(d + 2) * kPad + j] = q.z, sQ[(d + 3) * kPad + j] = q.w;
+    sK[d * kPad + j] = k.x, sK[(d + 1) * kPad + j] = k.y, sK[(d + 2) * kPad + j] = k.z, sK[(d + 3) * kPad + j] = k.w;
+  }
+  for (int i = tid; i < kChunk * v4; i += kThreads) {
+    const int j = i / v4, c = (i - j * v4) * 4;
+    *reinterpret_cast<float4*>(sV + j * a.vdimp + c) =
+        j < p.len ? *reinterpret_cast<const float4*>(vb + (size_t)j * a.ld + c) : make_float4(0, 0, 0, 0);
+  }
+  __syncthreads();
+  {
+    float s[4][4] = {};
+    tile_fma<1>(s, sQ, kPad, sK, kPad, a.dimp, ty, tx, 64);
+    __syncthreads();  // k is no longer needed
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+#pragma unroll
+      for (int r = 0; r < 4; ++r) {
+        const int i = ty * 4 + r, j = tx * 4 + c;
+        sA[j * kPad + i] = j <= i ? s[r][c] * pw[i - j] : 0.0f;
+      }
+  }
+  float acc[4][4 * NC] = {};
+  const float* S = a.chunk_state + ((size_t)chunk * a.heads + h) * a.dimp * a.vdimp;
+  for (int d0 = 0; d0 < a.dimp; d0 += kStateRows) {  // dimp is a multiple of 16
+    for (int i = tid; i < kStateRows * v4; i += kThreads)
+      reinterpret_cast<float4*>(sS)[i] = reinterpret_cast<const float4*>(S + (size_t)d0 * a.vdimp)[i];
+    __syncthreads();
+    tile_fma<NC>(acc, sQ + (size_t)d0 * kPad, kPad, sS, a.vdimp, kStateRows, ty, tx, a.vdimp);
+    __syncthreads();
+  }
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    const float f = pw[ty * 4 + r + 1];
+#pragma unroll
+    for (int i = 0; i < 4 * NC; ++i) acc[r][i] *= f;
+  }
+  tile_fma<NC>(acc, sA, kPad, sV, a.vdimp, min(p.len, ty / 2 * 8 + 8), ty, tx, a.vdimp);
+  T* out = static_cast<T*>(a.out);
+#pragma unroll
+  for (int r = 0; r < 4; ++r) {
+    float ss = 0.0f;
+#pragma unroll
+    for (int i = 0; i < 4 * NC; ++i) ss += acc[r][i] * acc[r][i];
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const int j = ty * 4 + r;
+    if (j >= p.len) continue;
+    const float inv = 1.0f / sqrtf(ss / (float)a.vdim + a.eps);
+#pragma unroll
+    for (int i = 0; i < NC; ++i) {
+      const int c = tx * 4 + i * 64;
+      if (c < a.vdimp) {
+        const float4 g = *reinterpret_cast<const float4*>(gb + (size_t)j * a.ld + c);
+        T* o = out + (size_t)(p.row0 + j) * a.ldo + h * a.vdimp + c;
+        o[0] = from_f32<T>(acc[r][4 * i] * inv * silu(g.x));
+        o[1] = from_f32<T>(acc[r][4 * i + 1] * inv * silu(g.y));
+        o[2] = from_f32<T>(acc[r][4 * i + 2] * inv * silu(g.z));
+        o[3] = from_f32<T>(acc[r][4 * i + 3] * inv * silu(g.w));
+      }
+    }
+  }
+}
+
+template <class T, int NC>
+cudaError_t prefill_nc(cudaStream_t s, const RetentionArgs& a) {
+  cudaError_t r = launch_pdl(lm_ret_rotate_kernel, dim3(a.rows), dim3(kThreads), 0, s, a);
+  if (r == cudaSuccess)
+    r = launch_pdl(lm_ret_chunk_kernel<NC>, dim3(a.n_chunks, a.heads, (a.dimp + 63) / 64), dim3(kThreads), (size_t)kChunk * (64 + a.vdimp) * 4, s, a);
+  if (r == cudaSuccess) {
+    const int n4 = a.dimp * a.vdimp / 4;
+    r = launch_pdl(lm_ret_scan_kernel, dim3((n4 + kThreads - 1) / kThreads, a.heads, a.n_entries), dim3(kThreads), 0, s, a);
+  }
+  if (r == cudaSuccess) r = launch_pdl(lm_ret_output_kernel<T, NC>, dim3(a.n_chunks, a.heads), dim3(kThreads), output_smem(a), s, a);
+  return r;
+}
+template <class T>
+cudaError_t prefill_t(cudaStream_t s, const RetentionArgs& a) {
+  return a.vdimp <= 64 ? prefill_nc<T, 1>(s, a) : a.vdimp <= 128 ? prefill_nc<T, 2>(s, a) : prefill_nc<T, 4>(s, a);
+}
+
+constexpr int kRetSmemMax = 220 * 1024;
+
+}  // namespace
+
+cudaError_t retention_configure() {
+  cudaError_t r = cudaSuccess;
+  auto set = [&](auto f) {
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, kRetSmemMax);
+  };
+  set(lm_ret_chunk_kernel<1>);
+  set(lm_ret_chunk_kernel<2>);
+  set(lm_ret_chunk_kernel<4>);
+  set(lm_ret_output_kernel<float, 1>);
+  set(lm_ret_output_kernel<float, 2>);
+  set(lm_ret_output_kernel<float, 4>);
+  set(lm_ret_output_kernel<__nv_bfloat16, 1>);
+  set(lm_ret_output_kernel<__nv_bfloat16, 2>);
+  set(lm_ret_output_kernel<__nv_bfloat16, 4>);
+  return r;
+}
+
+cudaError_t launch_rope_table(cudaStream_t s, float* cos_t, float* sin_t, int max_pos, int dims, double base) {
+  const int n = max_pos * (dims / 2);
+  if (n > 0) lm_rope_table_kernel<<<(n + 255) / 256, 256, 0, s>>>(cos_t, sin_t, max_pos, dims / 2, base);
+  return cudaGetLastError();
+}
+
+cudaError_t launch_retention_decode(cudaStream_t s, bool f32, const RetentionArgs& a) {
+  const int rg = kThreads / (a.vdimp / 4);
+  const size_t smem = ((size_t)2 * a.dimp + a.vdimp + (size_t)rg * a.vdimp) * 4;
+  const dim3 grid(a.heads, a.rows);
+  return f32 ? launch_pdl(lm_ret_decode_kernel<float>, grid, dim3(kThreads), smem, s, a)
+             : launch_pdl(lm_ret_decode_kernel<__nv_bfloat16>, grid, dim3(kThreads), smem, s, a);
+}
+cudaError_t launch_retention_prefill(cudaStream_t s, bool f32, const RetentionArgs& a) {
+  return f32 ? prefill_t<float>(s, a) : prefill_t<__nv_bfloat16>(s, a);
+}
+
+}  // namespace lm
+}  // namespace mllmb200

@@ -5,8 +5,6 @@
 
 namespace mllmb200 {
 
-__device__ unsigned int g_device_status = 0;
-
 // One thread per (row in shard, K-group): moves the group's 16 nibble bytes and its scale.
 __global__ void repack_cells_kernel(const uint8_t* __restrict__ nibbles, const uint16_t* __restrict__ scales,
                                     int k, int row_begin, int row_count, int num_groups, int num_panels,

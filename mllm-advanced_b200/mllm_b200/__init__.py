@@ -11,3 +11,5 @@ from .binding import (  # noqa: F401
     blob_sections, tiled_size, workspace_size, W4A32Weights, linear_forward, linear_forward_grouped, quant_activations, check_device_status, conv3d_forward,
 )
 from .decoder import Qwen2Decoder, Qwen2BatchDecoder, Qwen2Config, QWEN2_1P5B, LINEAR_NAMES, plan_check, DECODE_AUTO, DECODE_GRAPH, DECODE_PERSISTENT  # noqa: F401,E402
+from .lm import LanguageModel, EngineError  # noqa: F401,E402
+from . import registry, scheduler  # noqa: F401,E402
