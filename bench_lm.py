@@ -1,0 +1,212 @@
+"""`bench.py --lm`: prefill and decode throughput of the Vupuzen design on the language-model engine (random bf16 weights)
+beside the quantized Qwen2 decoder at equal layer sizes: same width, heads, head size, feed-forward, vocabulary and depth.
+Device times by CUDA events on the engines' streams; the best of a few repetitions.  Every timed step streams more
+weights than L2 holds (the smallest model reads 0.7 GB per step).
+
+Roofline: a prompt against the measured bf16 rate (dense products of the linears, causal attention, chunked retention), a
+decode step against the measured copy bandwidth (weights once, every cache and state byte once, states written too)."""
+import numpy as np
+
+SIZES = {
+    # layers like published models of this scale; every fourth layer is retention
+    "0.5b": dict(width=896, layers=24, heads=14, kv=2, dim=64, ff=4864, vocab=151936),
+    "1.5b": dict(width=1536, layers=28, heads=12, kv=2, dim=128, ff=8960, vocab=151936),
+    "2048": dict(width=2048, layers=16, heads=16, kv=4, dim=128, ff=8192, vocab=32000),
+}
+
+
+def build(torch, lm, s, max_seqs, max_ctx, max_rows, seed=0):
+    """A Vupuzen model of these sizes with random weights made on the device."""
+    gen = torch.Generator(device="cuda").manual_seed(seed)
+    W, H, G, D, F = s["width"], s["heads"], s["kv"], s["dim"], s["ff"]
+    layers = []
+    for i in range(s["layers"]):
+        base = dict(heads=H, dim=D, vdim=D, ff=F, ff_limit=7.0)
+        if i % 4 == 3:
+            layers.append(dict(base, mixer=lm.RETENTION, kv_heads=H, rot_dims=D, rot_base=1e6))
+        else:
+            layers.append(dict(base, mixer=lm.ATTENTION, kv_heads=G, score_scale=D ** -0.5, sink=1, bias_rows=32, bias_max=1024))
+    m = lm.LanguageModel(dict(vocab=s["vocab"], width=W, conv_taps=4, max_seqs=max_seqs, max_ctx=max_ctx, max_rows=max_rows, eps=1e-6,
+                              logit_scale=1.0), layers)
+    rand = lambda n, k: torch.randn((n, k), device="cuda", generator=gen).mul_(k ** -0.5).bfloat16()
+    emb = torch.randn((s["vocab"], W), device="cuda", generator=gen).bfloat16()
+    m.set_tensor(-1, "embed", emb)
+    m.set_tensor(-1, "head", emb[torch.randperm(s["vocab"], device="cuda", generator=gen)])  # greedy decoding walks a permutation
+    m.set_tensor(-1, "final_norm", np.float32(1))
+    for i, d in enumerate(layers):
+        attn = d["mixer"] == lm.ATTENTION
+        for name, n, k in [("q", H * D, W), ("k", d["kv_heads"] * D, W), ("v", d["kv_heads"] * D, W), ("o", W, H * D), ("gate", F, W),
+                           ("up", F, W), ("down", W, F)] + ([] if attn else [("g", H * D, W)]):
+            m.set_tensor(i, name, rand(n, k))
+        for name in ("norm1", "norm1b", "norm2", "norm2b"):
+            m.set_tensor(i, name, np.float32(0.25 if name.endswith("b") else 1))
+        m.set_tensor(i, "conv", np.random.default_rng(i).standard_normal((W, 4)).astype(np.float32) * 0.2)
+        if attn:
+            m.set_tensor(i, "rel", np.random.default_rng(i).standard_normal((32, H)).astype(np.float32) * 0.3)
+        else:
+            m.set_tensor(i, "decay", 1.0 - 2.0 ** -(5.0 + np.arange(H) * 8.0 / H))
+    return m
+
+
+def mixer_kinds(s):
+    ret = s["layers"] // 4
+    return s["layers"] - ret, ret
+
+
+def linear_weights(s):
+    """bf16 weights of all layers' linears, in elements."""
+    W, H, G, D, F = s["width"], s["heads"], s["kv"], s["dim"], s["ff"]
+    a, r = mixer_kinds(s)
+    return a * (W * D * (H + 2 * G) + W * H * D) + r * (4 * W * H * D + W * H * D) + s["layers"] * 3 * W * F
+
+
+def prefill_flops(s, n):
+    H, D = s["heads"], s["dim"]
+    a, r = mixer_kinds(s)
+    attn = a * 2 * 2 * H * D * n * (n + 1) / 2
+    ret = r * 2 * n * H * (2 * 64 / 2 * D + 2 * D * D)
+    return 2 * n * linear_weights(s) + attn + ret + 2 * s["vocab"] * s["width"]
+
+
+def decode_bytes(s, batch, ctx):
+    H, G, D = s["heads"], s["kv"], s["dim"]
+    a, r = mixer_kinds(s)
+    return 2 * linear_weights(s) + 2 * s["vocab"] * s["width"] + batch * (a * 2 * G * D * 2 * ctx + r * 2 * H * D * D * 4)
+
+
+def event_ms(torch, stream, fn):
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record(stream)
+    fn()
+    b.record(stream)
+    stream.synchronize()
+    return a.elapsed_time(b)
+
+
+def time_vupuzen(torch, lm, s, prompts, batches, ctx, steps, hbm, tflops):
+    rows = max(prompts)
+    m = build(torch, lm, s, max(batches), max(rows, ctx + steps + 8), rows)
+    st, rng, out = m.stream(), np.random.default_rng(1), {"prefill": {}, "decode": {}}
+    for n in prompts:
+        toks, ms = rng.integers(0, s["vocab"], n).tolist(), []
+        for _ in range(5):
+            slot = m.acquire()
+            ms.append(event_ms(torch, st, lambda: m.step([(slot, toks)], sample=True)))
+            m.release(slot)
+        t, f = min(ms[1:]), prefill_flops(s, n)
+        out["prefill"][n] = {"ms": t, "tokens_per_s": n / t * 1e3, "tflops": f / t / 1e9, "frac_bf16": f / t / 1e9 / tflops}
+    for b in batches:
+        slots = [m.acquire() for _ in range(b)]
+        for k, slot in enumerate(slots):
+            m.step([(slot, rng.integers(0, s["vocab"], ctx - 5 - k % 7).tolist())], sample=True)
+        m.decode(slots, 4)
+        ms = min(event_ms(torch, st, lambda: m.decode(slots, steps // 4)) for _ in range(4)) / (steps // 4)
+        distinct = len({tuple(m.read(x, ctx - 3, steps).tolist()) for x in slots})
+        by = decode_bytes(s, b, ctx + steps / 2)
+        out["decode"][b] = {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3, "context": ctx, "GBs": by / ms / 1e6,
+                            "frac_hbm": by / ms / 1e6 / hbm, "sequences_differ": distinct == b}
+        for slot in slots:
+            m.release(slot)
+    m.check_device_status()
+    m.close()
+    return out
+
+
+def time_qwen2(torch, mb, bench, s, prompts, batches, ctx, steps, hbm, tflops):
+    H, G, D, W, F = s["heads"], s["kv"], s["dim"], s["width"], s["ff"]
+    gen = torch.Generator(device="cuda").manual_seed(3)
+    cfg = dict(layers=s["layers"], hidden=W, q_heads=H, kv_heads=G, head_dim=D, inter=F, vocab=s["vocab"],
+               max_ctx=max(max(prompts) + 1, ctx + steps + 8), eps=1e-6, rope_theta=1e6)
+    dec = mb.Qwen2Decoder(cfg)
+    shapes = [("q", W, H * D, True), ("k", W, G * D, True), ("v", W, G * D, True), ("o", H * D, W, False), ("gate", W, F, False),
+              ("up", W, F, False), ("down", F, W, False)]
+    for i in range(s["layers"]):
+        for name, k, n, bias in shapes:
+            dec.set_linear_tiled(i, name, bench.make_random_weights(mb, torch, n, k, bias, gen))
+        dec.set_norm(0, i, np.ones(W, np.float32))
+        dec.set_norm(1, i, np.ones(W, np.float32))
+    dec.set_norm(2, 0, np.ones(W, np.float32))
+    emb = torch.randn((s["vocab"], W), device="cuda", generator=gen) * 16
+    dec.set_tables(emb, (emb * 0.02).half())
+    st, rng, out = dec.stream(), np.random.default_rng(1), {"prefill": {}, "decode": {}}
+    lin = s["layers"] * sum(n * k for _, k, n, _ in shapes)
+    for n in prompts:
+        toks = torch.from_numpy(rng.integers(0, s["vocab"], n).astype(np.int32)).cuda()
+        torch.cuda.synchronize()
+        t = min([event_ms(torch, st, lambda: dec.prefill_device(toks)) for _ in range(5)][1:])
+        f = 2 * n * lin + s["layers"] * 2 * H * D * n * (n + 1) + 2 * s["vocab"] * W
+        out["prefill"][n] = {"ms": t, "tokens_per_s": n / t * 1e3, "tflops": f / t / 1e9, "frac_bf16": f / t / 1e9 / tflops}
+
+    def entry(ms, b):
+        by = lin * 0.5625 + 2 * s["vocab"] * W + b * s["layers"] * 2 * G * D * 4 * (ctx + steps / 2)
+        return {"ms_per_step": ms, "tokens_per_s": b / ms * 1e3, "context": ctx, "GBs": by / ms / 1e6, "frac_hbm": by / ms / 1e6 / hbm}
+
+    for b in batches:
+        if b == 1:
+            dec.prefill(rng.integers(0, s["vocab"], ctx))
+            dec.decode(4)
+            ms = min(event_ms(torch, st, lambda: dec.decode(steps // 4)) for _ in range(4)) / (steps // 4)
+        else:
+            try:
+                bd = mb.Qwen2BatchDecoder(dec, b)
+            except mb.MllmB200Error:  # its batched lm_head holds the activations in shared memory: widths up to about 1700
+                out["decode"][b] = None
+                continue
+            bd.set_policy(5)
+            for k in range(b):
+                bd.prefill(k, tokens=rng.integers(0, s["vocab"], ctx))
+            bd.decode(4)
+            ms = min(event_ms(torch, st, lambda: bd.decode(steps // 4)) for _ in range(4)) / (steps // 4)
+            bd.close()
+        out["decode"][b] = entry(ms, b)
+    mb.check_device_status(st)
+    dec.close()
+    return out
+
+
+def once(torch, mb, bench, which, size, layers):
+    """A short untimed run for a profiler's launch list: one prompt, then a few decode steps."""
+    from mllm_b200 import lm
+    s = dict(SIZES[size], layers=layers, vocab=8192)
+    if which == "vupuzen":
+        m = build(torch, lm, s, 64, 1200, 2048)
+        rng = np.random.default_rng(0)
+        slots = [m.acquire() for _ in range(64)]
+        m.step([(slots[0], rng.integers(0, 8192, 1024).tolist())], sample=True)
+        for x in slots[1:]:
+            m.step([(x, rng.integers(0, 8192, 1024).tolist())], sample=True)
+        m.decode(slots, 1)
+        m.decode(slots[:1], 1)
+        m.synchronize()
+        m.check_device_status()
+        m.close()
+    else:
+        time_qwen2(torch, mb, bench, s, [1024], [1, 64], 1024, 4, 1.0, 1.0)
+
+
+def run(args, bench):
+    import torch
+    import mllm_b200 as mb
+    from mllm_b200 import lm
+    torch.cuda.set_device(0)
+    if args.lm_once:
+        once(torch, mb, bench, args.lm_once, args.lm_size or "1.5b", 4)
+        return {"once": args.lm_once}
+    hbm, tflops, kind = bench.measured_peaks()
+    prompts, batches, ctx, steps = [128, 512, 2048], [1, 8, 64], 512, 64
+    out = {"metric": "language-model engine, Vupuzen beside Qwen2 W4A32 at equal layer sizes", "unit": "tokens/s", "data": "synthetic",
+           "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tflops, "kind": kind}, "sizes": {}}
+    sampler = bench.ClockSampler(0)
+    sampler.start()
+    import time
+    t0 = time.time()
+    for name in [args.lm_size] if args.lm_size else SIZES:
+        s = SIZES[name]
+        out["sizes"][name] = {"config": s, "vupuzen": time_vupuzen(torch, lm, s, prompts, batches, ctx, steps, hbm, tflops)}
+        torch.cuda.empty_cache()
+        if not args.lm_no_compare:
+            out["sizes"][name]["qwen2_w4a32"] = time_qwen2(torch, mb, bench, s, prompts, batches, ctx, steps, hbm, tflops)
+            torch.cuda.empty_cache()
+    out["clocks"] = sampler.summary(t0, time.time())
+    sampler.stop()
+    return out

@@ -10,12 +10,12 @@ _NUMPY = {"F64": np.float64, "F32": np.float32, "F16": np.float16, "I64": np.int
 
 
 def bf16_to_f32(bits):
-    return (np.asarray(bits, np.uint16).astype(np.uint32) << 16).view(np.float32)
+    return (np.asarray(bits, np.uint16).astype(np.uint32) << 16).view(np.float32)  # (a scalar for a tensor of no dimensions)
 
 
 def f32_to_bf16(x):
     """Bits of the nearest bf16 (ties to even) of finite numbers."""
-    u = np.ascontiguousarray(x, np.float32).view(np.uint32)
+    u = np.asarray(x, np.float32).view(np.uint32)
     return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
 
 
@@ -67,7 +67,7 @@ def save(path, tensors):
     """Writes {name: (dtype name, array)} (bf16 as uint16 bits)."""
     header, blobs, at = {}, [], 0
     for name, (dt, a) in tensors.items():
-        b = np.ascontiguousarray(a).tobytes()
+        b = np.asarray(a).tobytes()
         header[name] = {"dtype": dt, "shape": list(np.shape(a)), "data_offsets": [at, at + len(b)]}
         blobs.append(b)
         at += len(b)
