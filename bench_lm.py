@@ -169,19 +169,19 @@ def once(torch, mb, bench, which, size, layers):
     from mllm_b200 import lm
     s = dict(SIZES[size], layers=layers, vocab=8192)
     if which == "vupuzen":
-        m = build(torch, lm, s, 64, 1200, 2048)
+        m = build(torch, lm, s, 64, 1200, 16384)
         rng = np.random.default_rng(0)
         slots = [m.acquire() for _ in range(64)]
         m.step([(slots[0], rng.integers(0, 8192, 1024).tolist())], sample=True)
-        for x in slots[1:]:
-            m.step([(x, rng.integers(0, 8192, 1024).tolist())], sample=True)
+        for k in range(1, 64, 16):
+            m.step([(x, rng.integers(0, 8192, 1024).tolist()) for x in slots[k:k + 16]], sample=True)
         m.decode(slots, 1)
         m.decode(slots[:1], 1)
         m.synchronize()
         m.check_device_status()
         m.close()
     else:
-        time_qwen2(torch, mb, bench, s, [1024], [1, 64], 1024, 4, 1.0, 1.0)
+        time_qwen2(torch, mb, bench, s, [1024], [1], 1024, 4, 1.0, 1.0)
 
 
 def run(args, bench):

@@ -5,7 +5,8 @@
 // fp32 and feed the weights to the value product as a sum of two bf16 numbers.
 //   * lm_attn_prefill_kernel: tiles of 64 (token, head) rows that share a kv head, key blocks of 64 through a
 //     double-buffered cp.async ring, mma.sync m16n8k16, online softmax in registers.
-//   * lm_attn_decode_kernel + lm_attn_combine_kernel: one token per sequence, the context split over CTAs.
+//   * lm_attn_decode_kernel + lm_attn_combine_kernel: one token per sequence, the context split over CTAs in chunks of 64
+//     or 128 positions, the query heads of a kv head as the rows of one mma tile.
 //   * lm_attn_f32_kernel: the 32-bit mode, any step.
 #include <algorithm>
 
@@ -274,26 +275,18 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
 }
 
 // ------------------------------------------------------------------------------------------ bf16 decode
-constexpr int kDecThreads = 128, kDecLanes = 8, kDecPass = kDecThreads / kDecLanes, kDecUnroll = 4;
+constexpr int kDecThreads = 128, kDecWarps = 4, kDecRows = 16;  // query heads per CTA: the rows of one mma tile
 
-__device__ __forceinline__ void unpack8(const uint4& p, float (&f)[8]) {
-  const uint32_t w[4] = {p.x, p.y, p.z, p.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    f[2 * i] = __uint_as_float(w[i] << 16);
-    f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-  }
+size_t decode_smem(const AttnShape& a, int chunk) {
+  const size_t tiles = (size_t)chunk * (a.dimp + 8 + a.vdimp + 8) * 2, merge = (size_t)kDecWarps * kDecRows * a.vdimp * 4;
+  return (size_t)kDecRows * (a.dimp + 8) * 2 + std::max(tiles, merge);
 }
 
-size_t decode_smem(const AttnShape& a, int hb) {
-  const int kg = kDecThreads / (a.vdimp / 8);
-  return ((size_t)hb * a.dimp + (size_t)hb * kDecodeKeys + (size_t)kg * hb * a.vdimp) * 4;
-}
-
-// grid (splits, kv heads x blocks of HB query heads, single rows).  One chunk of kDecodeKeys cache positions: scores
-// (eight lanes per key, 16-byte loads), softmax of the chunk, values (lanes over the value vector, the rest of the CTA
-// over keys).  splits == 1: the result; else {max, sum} and the unnormalized output per split.
-template <int HB>
+// grid (splits, kv heads x blocks of 16 query heads, single rows).  A CTA takes WK x 64 cache positions: all of their
+// keys and values are requested at once, each warp multiplies WK x 16 of them with the block's query heads, and the
+// warps' online-softmax states meet in shared memory.  One split: the result; else {max, sum} (base 2) and the
+// unnormalized output per split.
+template <int DV, int WK>
 __global__ void __launch_bounds__(kDecThreads) lm_attn_decode_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, int ldq,
                                                                      const int* __restrict__ single_rows,
                                                                      const int2* __restrict__ row_sp,
@@ -301,156 +294,193 @@ __global__ void __launch_bounds__(kDecThreads) lm_attn_decode_kernel(AttnShape a
                                                                      const __nv_bfloat16* __restrict__ vc,
                                                                      const float* __restrict__ bias, __nv_bfloat16* __restrict__ out,
                                                                      int ldo, float* __restrict__ part_o, float2* __restrict__ part_ml) {
-  extern __shared__ __align__(16) float dec_smem[];
-  __shared__ float s_m[HB], s_l[HB];
+  extern __shared__ __align__(16) uint8_t dec_smem[];
+  __shared__ float s_m[kDecWarps][kDecRows], s_l[kDecWarps][kDecRows];
+  constexpr int kKeys = 64 * WK;
   pdl_launch_dependents();
   pdl_wait_prior();
-  const int D = a.dimp, DV = a.vdimp, group = a.heads / a.kv_heads, hblocks = (group + HB - 1) / HB;
-  float* sq = dec_smem;                 // [HB][D]
-  float* ss = sq + HB * D;              // [HB][kDecodeKeys]
-  float* red = ss + HB * kDecodeKeys;   // [key groups][HB][DV]
-  const int split = blockIdx.x, splits = gridDim.x, kvh = blockIdx.y / hblocks, hb0 = (blockIdx.y - kvh * hblocks) * HB;
+  const int D = a.dimp, group = a.heads / a.kv_heads, hblocks = (group + kDecRows - 1) / kDecRows;
+  const int ldk = D + 8, ldv = a.vdimp + 8;
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(dec_smem);
+  __nv_bfloat16* sK = sQ + kDecRows * ldk;
+  __nv_bfloat16* sV = sK + kKeys * ldk;
+  float* sO = reinterpret_cast<float*>(sK);  // [warps][rows][vdimp], once keys and values are used up
+  const int split = blockIdx.x, splits = gridDim.x, kvh = blockIdx.y / hblocks, hb0 = (blockIdx.y - kvh * hblocks) * kDecRows;
   const int idx = blockIdx.z, row = single_rows ? single_rows[idx] : idx;
   const int2 sp = row_sp[row];
-  const int j0 = split * kDecodeKeys, nk = min(kDecodeKeys, sp.y + 1 - j0);
+  const int j0 = split * kKeys, nk = min(kKeys, sp.y + 1 - j0);
   if (nk <= 0) return;
-  const int nh = min(HB, group - hb0), h0 = kvh * group + hb0, tid = threadIdx.x;
+  const int nh = min(kDecRows, group - hb0), h0 = kvh * group + hb0, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const size_t base = ((size_t)sp.x * a.kv_heads + kvh) * a.max_ctx + j0;
-  for (int i = tid; i < HB * D; i += kDecThreads)
-    sq[i] = i / D < nh ? __bfloat162float(q[(size_t)row * ldq + h0 * D + i]) : 0.0f;
-  __syncthreads();
-  {
-    const int kl = tid / kDecLanes, l = tid % kDecLanes, vecs = D / 8;
-    for (int k0 = 0; k0 < nk; k0 += kDecPass * kDecUnroll) {
-      float acc[kDecUnroll][HB];
-#pragma unroll
-      for (int u = 0; u < kDecUnroll; ++u)
-#pragma unroll
-        for (int h = 0; h < HB; ++h) acc[u][h] = 0.0f;
-      for (int v = l; v < vecs; v += kDecLanes) {
-        uint4 raw[kDecUnroll];
-#pragma unroll
-        for (int u = 0; u < kDecUnroll; ++u) {
-          const int k = k0 + u * kDecPass + kl;
-          raw[u] = k < nk ? *reinterpret_cast<const uint4*>(kc + (base + k) * D + v * 8) : make_uint4(0, 0, 0, 0);
-        }
-        float kf[kDecUnroll][8];
-#pragma unroll
-        for (int u = 0; u < kDecUnroll; ++u) unpack8(raw[u], kf[u]);
-#pragma unroll
-        for (int h = 0; h < HB; ++h) {
-          const float4 qa = *reinterpret_cast<const float4*>(sq + h * D + v * 8), qb = *reinterpret_cast<const float4*>(sq + h * D + v * 8 + 4);
-          const float qv[8] = {qa.x, qa.y, qa.z, qa.w, qb.x, qb.y, qb.z, qb.w};
-#pragma unroll
-          for (int u = 0; u < kDecUnroll; ++u)
-#pragma unroll
-            for (int e = 0; e < 8; ++e) acc[u][h] = fmaf(qv[e], kf[u][e], acc[u][h]);
-        }
-      }
-#pragma unroll
-      for (int u = 0; u < kDecUnroll; ++u)
-#pragma unroll
-        for (int h = 0; h < HB; ++h) {
-#pragma unroll
-          for (int o = kDecLanes / 2; o > 0; o >>= 1) acc[u][h] += __shfl_xor_sync(0xffffffffu, acc[u][h], o);
-          const int k = k0 + u * kDecPass + kl;
-          if (l == h % kDecLanes && h < nh && k < nk) {
-            float s = acc[u][h] * a.scale;
-            if (a.has_bias) s += __ldg(bias + (size_t)(h0 + h) * (a.bias_max + 1) + min(sp.y - (j0 + k), a.bias_max));
-            ss[h * kDecodeKeys + k] = s;
-          }
-        }
-    }
+  const int dv8 = D / 8, vv8 = a.vdimp / 8;
+  for (int i = tid; i < kDecRows * dv8; i += kDecThreads) {
+    const int r = i / dv8, c = i - r * dv8;
+    cp_async16(smem_u32(sQ + r * ldk + c * 8), q + (size_t)row * ldq + (size_t)(h0 + (r < nh ? r : 0)) * D + c * 8, r < nh);
   }
-  __syncthreads();
-  for (int h = tid >> 5; h < nh; h += kDecThreads / 32) {
-    const int lane = tid & 31;
-    float mx = a.sink && splits == 1 ? 0.0f : kNegInf;
-    for (int k = lane; k < nk; k += 32) mx = fmaxf(mx, ss[h * kDecodeKeys + k]);
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    float sum = 0.0f;
-    for (int k = lane; k < nk; k += 32) {
-      const float p = expf(ss[h * kDecodeKeys + k] - mx);
-      ss[h * kDecodeKeys + k] = p;
-      sum += p;
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-    if (lane == 0) {
-      s_m[h] = mx;
-      s_l[h] = sum + (a.sink && splits == 1 ? expf(-mx) : 0.0f);
-    }
+  for (int i = tid; i < kKeys * dv8; i += kDecThreads) {
+    const int r = i / dv8, c = i - r * dv8;
+    cp_async16(smem_u32(sK + r * ldk + c * 8), kc + (base + (r < nk ? r : 0)) * D + c * 8, r < nk);
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  for (int i = tid; i < kKeys * vv8; i += kDecThreads) {
+    const int r = i / vv8, c = i - r * vv8;
+    cp_async16(smem_u32(sV + r * ldv + c * 8), vc + (base + (r < nk ? r : 0)) * a.vdimp + c * 8, r < nk);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const int k0 = warp * 16 * WK, mat = lane >> 3, ml = lane & 7;
+  float s[2 * WK][4], m[2] = {kNegInf, kNegInf}, l[2] = {0.0f, 0.0f}, o[DV / 8][4];
+#pragma unroll
+  for (int n = 0; n < 2 * WK; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {  // the bias (base 2), while the keys are on their way
+      const int hr = (lane >> 2) + (i >> 1) * 8, dist = sp.y - (j0 + k0 + n * 8 + (lane & 3) * 2 + (i & 1));
+      s[n][i] = a.has_bias && hr < nh && dist >= 0 ? kLog2e * __ldg(bias + (size_t)(h0 + hr) * (a.bias_max + 1) + min(dist, a.bias_max)) : 0.0f;
+    }
+#pragma unroll
+  for (int n = 0; n < DV / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
+  asm volatile("cp.async.wait_group 1;" ::: "memory");
   __syncthreads();
-  const int vl_n = DV / 8, kg_n = kDecThreads / vl_n, vl = tid % vl_n, kg = tid / vl_n;
-  if (kg < kg_n) {
-    float acc[HB][8];
+  if (k0 < nk) {
+    const uint32_t q_addr = smem_u32(sQ + ((mat & 1) * 8 + ml) * ldk + (mat >> 1) * 8);
+    const uint32_t k_addr = smem_u32(sK + (k0 + (mat >> 1) * 8 + ml) * ldk + (mat & 1) * 8);
+    float acc[2 * WK][4] = {};
+    for (int kk = 0; kk < D; kk += 16) {
+      uint32_t qa[4];
+      ldsm4(qa, q_addr + kk * 2);
 #pragma unroll
-    for (int h = 0; h < HB; ++h)
-#pragma unroll
-      for (int e = 0; e < 8; ++e) acc[h][e] = 0.0f;
-    for (int k0 = kg; k0 < nk; k0 += kg_n * kDecUnroll) {
-      uint4 raw[kDecUnroll];
-#pragma unroll
-      for (int u = 0; u < kDecUnroll; ++u) {
-        const int k = k0 + u * kg_n;
-        raw[u] = k < nk ? *reinterpret_cast<const uint4*>(vc + (base + k) * DV + vl * 8) : make_uint4(0, 0, 0, 0);
-      }
-#pragma unroll
-      for (int u = 0; u < kDecUnroll; ++u) {
-        const int k = k0 + u * kg_n;
-        if (k >= nk) break;
-        float vf[8];
-        unpack8(raw[u], vf);
-#pragma unroll
-        for (int h = 0; h < HB; ++h) {
-          const float p = h < nh ? ss[h * kDecodeKeys + k] : 0.0f;
-#pragma unroll
-          for (int e = 0; e < 8; ++e) acc[h][e] = fmaf(p, vf[e], acc[h][e]);
-        }
+      for (int n = 0; n < WK; ++n) {
+        uint32_t b[4];
+        ldsm4(b, k_addr + (n * 16 * ldk + kk) * 2);
+        mma_bf16(acc[2 * n], qa, b[0], b[1]);
+        mma_bf16(acc[2 * n + 1], qa, b[2], b[3]);
       }
     }
+    const float sc2 = a.scale * kLog2e;
 #pragma unroll
-    for (int h = 0; h < HB; ++h) {
-      float* r = red + ((size_t)kg * HB + h) * DV + vl * 8;
-      *reinterpret_cast<float4*>(r) = make_float4(acc[h][0], acc[h][1], acc[h][2], acc[h][3]);
-      *reinterpret_cast<float4*>(r + 4) = make_float4(acc[h][4], acc[h][5], acc[h][6], acc[h][7]);
+    for (int n = 0; n < 2 * WK; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int c = k0 + n * 8 + (lane & 3) * 2 + (i & 1);
+        s[n][i] = c < nk ? fmaf(acc[n][i], sc2, s[n][i]) : kNegInf;
+        m[i >> 1] = fmaxf(m[i >> 1], s[n][i]);
+      }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      m[r] = fmaxf(m[r], __shfl_xor_sync(0xffffffffu, m[r], 1));
+      m[r] = fmaxf(m[r], __shfl_xor_sync(0xffffffffu, m[r], 2));
+    }
+#pragma unroll
+    for (int n = 0; n < 2 * WK; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        s[n][i] = s[n][i] == kNegInf ? 0.0f : exp2f(s[n][i] - m[i >> 1]);
+        l[i >> 1] += s[n][i];
+      }
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
+      l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  if (k0 < nk) {
+    const uint32_t v_addr = smem_u32(sV + (k0 + (mat & 1) * 8 + ml) * ldv + (mat >> 1) * 8);
+#pragma unroll
+    for (int kk = 0; kk < WK; ++kk) {
+      uint32_t hi[4], lo[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float p0 = s[2 * kk + (i >> 1)][(i & 1) * 2], p1 = s[2 * kk + (i >> 1)][(i & 1) * 2 + 1];
+        hi[i] = pack2(p0, p1);
+        lo[i] = pack2(p0 - __uint_as_float(hi[i] << 16), p1 - __uint_as_float(hi[i] & 0xffff0000u));
+      }
+#pragma unroll
+      for (int n = 0; n < DV / 16; ++n)
+        if (n * 16 < a.vdimp) {
+          uint32_t b[4];
+          ldsm4_t(b, v_addr + (kk * 16 * ldv + n * 16) * 2);
+          mma_bf16(o[2 * n], hi, b[0], b[1]);
+          mma_bf16(o[2 * n], lo, b[0], b[1]);
+          mma_bf16(o[2 * n + 1], hi, b[2], b[3]);
+          mma_bf16(o[2 * n + 1], lo, b[2], b[3]);
+        }
     }
   }
   __syncthreads();
-  for (int i = tid; i < nh * DV; i += kDecThreads) {
-    float o = 0.0f;
-    for (int g = 0; g < kg_n; ++g) o += red[(size_t)g * HB * DV + i];
-    const int h = i / DV;
-    if (splits == 1) out[(size_t)row * ldo + h0 * DV + i] = __float2bfloat16_rn(o / s_l[h]);
-    else part_o[(((size_t)idx * a.heads + h0 + h) * splits + split) * DV + (i - h * DV)] = o;
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int hr = (lane >> 2) + r * 8;
+    if ((lane & 3) == 0) s_m[warp][hr] = m[r], s_l[warp][hr] = l[r];
+    float* so = sO + ((size_t)warp * kDecRows + hr) * a.vdimp + (lane & 3) * 2;
+#pragma unroll
+    for (int n = 0; n < DV / 8; ++n)
+      if (n * 8 < a.vdimp) *reinterpret_cast<float2*>(so + n * 8) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
   }
-  if (splits > 1 && tid < nh) part_ml[((size_t)idx * a.heads + h0 + tid) * splits + split] = make_float2(s_m[tid], s_l[tid]);
+  __syncthreads();
+  const bool whole = splits == 1;
+  for (int i = tid; i < nh * a.vdimp; i += kDecThreads) {
+    const int h = i / a.vdimp;
+    float mx = whole && a.sink ? 0.0f : kNegInf, sum, v = 0.0f;
+#pragma unroll
+    for (int w = 0; w < kDecWarps; ++w) mx = fmaxf(mx, s_m[w][h]);
+    sum = whole && a.sink ? exp2f(-mx) : 0.0f;
+#pragma unroll
+    for (int w = 0; w < kDecWarps; ++w) {
+      const float f = exp2f(s_m[w][h] - mx);
+      sum = fmaf(f, s_l[w][h], sum);
+      v = fmaf(f, sO[(size_t)w * kDecRows * a.vdimp + i], v);
+    }
+    if (whole) {
+      out[(size_t)row * ldo + h0 * a.vdimp + i] = __float2bfloat16_rn(v / sum);
+    } else {
+      const size_t at = ((size_t)idx * a.heads + h0 + h) * splits + split;
+      part_o[at * a.vdimp + (i - h * a.vdimp)] = v;
+      if (i == h * a.vdimp) part_ml[at] = make_float2(mx, sum);
+    }
+  }
 }
 
 // grid (heads, single rows): merges the splits of a row and head, the sink joining here.
-__global__ void __launch_bounds__(128) lm_attn_combine_kernel(AttnShape a, int splits, const int* __restrict__ single_rows,
+__global__ void __launch_bounds__(128) lm_attn_combine_kernel(AttnShape a, int chunk, int splits, const int* __restrict__ single_rows,
                                                               const int2* __restrict__ row_sp, const float* __restrict__ part_o,
                                                               const float2* __restrict__ part_ml, __nv_bfloat16* __restrict__ out,
                                                               int ldo) {
   extern __shared__ float sw[];  // [splits]
+  __shared__ float s_inv;
   pdl_launch_dependents();
   pdl_wait_prior();
   const int h = blockIdx.x, idx = blockIdx.y, row = single_rows ? single_rows[idx] : idx, tid = threadIdx.x;
-  const int nact = min(splits, row_sp[row].y / kDecodeKeys + 1);
+  const int nact = min(splits, row_sp[row].y / chunk + 1);
   const float2* ml = part_ml + ((size_t)idx * a.heads + h) * splits;
-  float mx = a.sink ? 0.0f : kNegInf;
-  for (int s = 0; s < nact; ++s) mx = fmaxf(mx, ml[s].x);
-  for (int s = tid; s < nact; s += blockDim.x) sw[s] = expf(ml[s].x - mx);
+  if (tid < 32) {
+    float mx = a.sink ? 0.0f : kNegInf;
+    for (int s = tid; s < nact; s += 32) mx = fmaxf(mx, ml[s].x);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+    float tot = 0.0f;
+    for (int s = tid; s < nact; s += 32) {
+      const float2 v = ml[s];
+      const float f = exp2f(v.x - mx);
+      sw[s] = f;
+      tot = fmaf(v.y, f, tot);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) tot += __shfl_xor_sync(0xffffffffu, tot, o);
+    if (tid == 0) s_inv = 1.0f / (tot + (a.sink ? exp2f(-mx) : 0.0f));
+  }
   __syncthreads();
-  float tot = a.sink ? expf(-mx) : 0.0f;
-  for (int s = 0; s < nact; ++s) tot = fmaf(ml[s].y, sw[s], tot);
-  const float inv = 1.0f / tot;
+  const float inv = s_inv;
   for (int d = tid; d < a.vdimp; d += blockDim.x) {
     const float* po = part_o + ((size_t)idx * a.heads + h) * splits * a.vdimp + d;
     float o = 0.0f;
-    for (int s = 0; s < nact; ++s) o = fmaf(sw[s], po[(size_t)s * a.vdimp], o);
+    for (int s0 = 0; s0 < nact; s0 += 8) {  // eight partial rows requested together
+      float v[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] = po[(size_t)min(s0 + j, nact - 1) * a.vdimp];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) o = fmaf(s0 + j < nact ? sw[s0 + j] : 0.0f, v[j], o);
+    }
     out[(size_t)row * ldo + h * a.vdimp + d] = __float2bfloat16_rn(o * inv);
   }
 }
@@ -469,10 +499,12 @@ cudaError_t attention_configure() {
   set(lm_attn_prefill_kernel<64>);
   set(lm_attn_prefill_kernel<128>);
   set(lm_attn_prefill_kernel<256>);
-  set(lm_attn_decode_kernel<1>);
-  set(lm_attn_decode_kernel<2>);
-  set(lm_attn_decode_kernel<4>);
-  set(lm_attn_decode_kernel<8>);
+  set(lm_attn_decode_kernel<64, 1>);
+  set(lm_attn_decode_kernel<64, 2>);
+  set(lm_attn_decode_kernel<128, 1>);
+  set(lm_attn_decode_kernel<128, 2>);
+  set(lm_attn_decode_kernel<256, 1>);
+  set(lm_attn_decode_kernel<256, 2>);
   return r;
 }
 
@@ -480,7 +512,7 @@ cudaError_t attention_configure() {
 // decode kernels; in 32-bit mode all `rows` rows take one kernel.
 cudaError_t launch_attention(cudaStream_t s, bool f32, const AttnShape& a, const void* q, int ldq, const int2* row_sp, int rows,
                              const void* kc, const void* vc, const float* bias, void* out, int ldo, const int4* tiles, int n_tiles,
-                             const int* single_rows, int n_single, int splits, float* part_o, float2* part_ml) {
+                             const int* single_rows, int n_single, int chunk, int splits, float* part_o, float2* part_ml) {
   if (f32)
     return launch_pdl(lm_attn_f32_kernel, dim3(rows, a.heads), dim3(kF32Threads), 0, s, a, static_cast<const float*>(q), ldq, row_sp,
                       static_cast<const float*>(kc), static_cast<const float*>(vc), bias, static_cast<float*>(out), ldo);
@@ -498,14 +530,16 @@ cudaError_t launch_attention(cudaStream_t s, bool f32, const AttnShape& a, const
   }
   if (n_single) {
     const int group = a.heads / a.kv_heads;
-    const int hb = group <= 1 ? 1 : group <= 2 ? 2 : group <= 4 ? 4 : 8;
-    const dim3 grid(splits, a.kv_heads * ((group + hb - 1) / hb), n_single);
-    const size_t smem = decode_smem(a, hb);
+    const dim3 grid(splits, a.kv_heads * ((group + kDecRows - 1) / kDecRows), n_single);
+    const size_t smem = decode_smem(a, chunk);
     auto go = [&](auto f) { return launch_pdl(f, grid, dim3(kDecThreads), smem, s, a, qb, ldq, single_rows, row_sp, kb, vb, bias, ob, ldo, part_o, part_ml); };
-    r = hb == 1 ? go(lm_attn_decode_kernel<1>) : hb == 2 ? go(lm_attn_decode_kernel<2>) : hb == 4 ? go(lm_attn_decode_kernel<4>) : go(lm_attn_decode_kernel<8>);
+    const bool two = chunk == 128;
+    r = a.vdimp <= 64    ? (two ? go(lm_attn_decode_kernel<64, 2>) : go(lm_attn_decode_kernel<64, 1>))
+        : a.vdimp <= 128 ? (two ? go(lm_attn_decode_kernel<128, 2>) : go(lm_attn_decode_kernel<128, 1>))
+                         : (two ? go(lm_attn_decode_kernel<256, 2>) : go(lm_attn_decode_kernel<256, 1>));
     if (r == cudaSuccess && splits > 1)
-      r = launch_pdl(lm_attn_combine_kernel, dim3(a.heads, n_single), dim3(128), (size_t)splits * 4, s, a, splits, single_rows, row_sp,
-                     part_o, part_ml, ob, ldo);
+      r = launch_pdl(lm_attn_combine_kernel, dim3(a.heads, n_single), dim3(128), (size_t)splits * 4, s, a, chunk, splits, single_rows,
+                     row_sp, part_o, part_ml, ob, ldo);
   }
   return r;
 }

@@ -24,9 +24,13 @@ namespace {
 constexpr int kArgmaxBlocks = 32;
 
 struct GraphKey {
-  int count, splits;
-  bool operator<(const GraphKey& o) const { return std::tie(count, splits) < std::tie(o.count, o.splits); }
+  int count, chunk, splits;
+  bool operator<(const GraphKey& o) const { return std::tie(count, chunk, splits) < std::tie(o.count, o.chunk, o.splits); }
 };
+// Positions per CTA of the decode attention: small pieces while they are needed to fill the GPU.
+int decode_chunk(int sequences, int longest) {
+  return (long long)sequences * ((longest + 127) / 128) >= 2 * kSms ? 128 : kMinDecodeChunk;
+}
 struct Graph {
   cudaGraphExec_t exec;
   long long launches;
@@ -41,7 +45,7 @@ struct StepCtx {
   bool single = false;  // one token per entry, row r = entry r
   // mixed steps: rows of one-token entries, prompt tiles per head-group size, retention chunks
   const int* single_rows = nullptr;
-  int n_single = 0, splits = 1;
+  int n_single = 0, chunk = kMinDecodeChunk, splits = 1;  // context split of the decode attention
   std::map<int, std::pair<const int4*, int>> tiles;
   const int2 *chunks = nullptr, *entry_chunks = nullptr;
   int n_chunks = 0;
@@ -185,7 +189,7 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
   const size_t rows = c.max_rows, slots = c.max_seqs;
   e->plane_rows = std::max(c.max_rows, 1024);
   e->logit_rows = std::max(std::min(c.max_rows, 128), c.max_seqs);
-  e->max_splits_ctx = (c.max_ctx + kDecodeKeys - 1) / kDecodeKeys;
+  e->max_splits_ctx = (c.max_ctx + kMinDecodeChunk - 1) / kMinDecodeChunk;
   LM_OK(dalloc(e, &e->embed, (size_t)c.vocab * c.width));
   LM_OK(make_linear(e, &e->head, c.vocab, c.width));
   LM_OK(dalloc(e, &e->final_gain, 1));
@@ -534,7 +538,7 @@ int mixer(Engine* e, const StepCtx& t, LayerState& L) {
     const int4* tiles = it == t.tiles.end() ? nullptr : it->second.first;
     const int n_tiles = it == t.tiles.end() ? 0 : it->second.second;
     LM_CUDA(launch_attention(e->stream, e->f32, s, e->proj, p.ldq, t.row_sp, t.rows, L.kc, L.vc, w.bias, e->mix, ldo, tiles, n_tiles,
-                             t.single ? nullptr : t.single_rows, t.single ? t.rows : t.n_single, t.splits, e->part_o, e->part_ml));
+                             t.single ? nullptr : t.single_rows, t.single ? t.rows : t.n_single, t.chunk, t.splits, e->part_o, e->part_ml));
     return MLLMB200_OK;
   }
   p.kind = kEpiPlanes;
@@ -741,7 +745,8 @@ int step(Engine* e, int n_entries, const int* slots, const int* counts, const in
   t.single = all_single;
   t.single_rows = d + o_sr;
   t.n_single = (int)single_rows.size();
-  t.splits = max_single / kDecodeKeys + 1;
+  t.chunk = decode_chunk(t.n_single, max_single + 1);
+  t.splits = max_single / t.chunk + 1;
   for (auto& g : tiles) t.tiles[g.first] = {reinterpret_cast<const int4*>(d + o_tiles[g.first]), (int)g.second.size()};
 
   const long long before = g_launches;
@@ -769,7 +774,7 @@ int step(Engine* e, int n_entries, const int* slots, const int* counts, const in
   return MLLMB200_OK;
 }
 
-int enqueue_decode(Engine* e, int count, int splits) {
+int enqueue_decode(Engine* e, int count, int chunk, int splits) {
   StepCtx t;
   t.rows = t.entries = count;
   t.tokens = e->d_row_token;
@@ -777,6 +782,7 @@ int enqueue_decode(Engine* e, int count, int splits) {
   t.row_entry = e->d_row_entry;
   t.entry = e->d_entries;
   t.single = true;
+  t.chunk = chunk;
   t.splits = splits;
   LM_CUDA(launch_decode_prep(e->stream, count, e->d_slots, e->d_pos, e->d_token, e->d_tail, e->d_row_sp, e->d_row_token, e->d_entries, e->d_row_entry));
   Stream r{};
@@ -804,15 +810,16 @@ int decode(Engine* e, int count, const int* slots, int steps) {
     e->cur_slots = now;
   }
   for (int i = 0; i < steps; ++i, ++longest) {
+    const int chunk = decode_chunk(count, longest + 1);
     int splits = 1;  // one graph per power of two of context chunks
-    while (splits * kDecodeKeys < longest + 1) splits *= 2;
-    splits = std::min(splits, e->max_splits_ctx);
-    auto it = e->graphs.find({count, splits});
+    while (splits * chunk < longest + 1) splits *= 2;
+    splits = std::min(splits, (c.max_ctx + chunk - 1) / chunk);
+    auto it = e->graphs.find({count, chunk, splits});
     if (it == e->graphs.end()) {
       const long long before = g_launches;
       cudaGraph_t g = nullptr;
       LM_CUDA(cudaStreamBeginCapture(e->stream, cudaStreamCaptureModeThreadLocal));
-      const int st = enqueue_decode(e, count, splits);
+      const int st = enqueue_decode(e, count, chunk, splits);
       const cudaError_t r = cudaStreamEndCapture(e->stream, &g);
       Graph gr{nullptr, g_launches - before};
       if (st == MLLMB200_OK && r == cudaSuccess) {
@@ -824,7 +831,7 @@ int decode(Engine* e, int count, const int* slots, int steps) {
         LM_OK(st);
         LM_CUDA(r);
       }
-      it = e->graphs.emplace(GraphKey{count, splits}, gr).first;
+      it = e->graphs.emplace(GraphKey{count, chunk, splits}, gr).first;
     }
     LM_CUDA(cudaGraphLaunch(it->second.exec, e->stream));
     e->launches += it->second.launches;

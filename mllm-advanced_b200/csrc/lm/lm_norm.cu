@@ -130,6 +130,129 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
   }
 }
 
+// The same for many rows: a warp per row for the sums (no block barrier inside), then - with a convolution - the threads
+// sweep the CTA's rows column by column with the last TW - 1 rows of h in registers.  x' of the CTA's own rows is read
+// back from x_out (or x_in when there is nothing to fold in), that of the rows in front of them from shared memory.
+constexpr int kManyRows = 16, kNormWarps = kNormThreads / 32;
+
+template <class T, int NVW, int TW>
+__global__ void __launch_bounds__(kNormThreads) lm_norm_rows_kernel(NormArgs a) {
+  extern __shared__ __align__(16) float halo[];  // [TW - 1][ldx]
+  __shared__ float s_r[kManyRows + 8];
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nv = a.ldx >> 2;
+  const float g_pre = *a.g_pre, g_post = a.delta ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
+  const int r_begin = blockIdx.x * kManyRows, r_end = min(r_begin + kManyRows, a.rows);
+  int t0 = r_begin;
+  if (TW > 1) t0 = max(r_begin - (a.taps - 1), a.entries[a.row_entry[r_begin]].row0);
+  auto warp_sum = [](float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+  };
+  for (int t = t0 + warp; t < r_end; t += kNormWarps) {
+    const float4* xr = reinterpret_cast<const float4*>(a.x_in + (size_t)t * a.ldx);
+    float4 x[NVW];
+    float ss = 0.0f;
+    if (a.delta) {
+      const float4* dr = reinterpret_cast<const float4*>(a.delta + (size_t)t * a.ldx);
+#pragma unroll
+      for (int i = 0; i < NVW; ++i) {
+        const int c = lane + i * 32;
+        x[i] = c < nv ? dr[c] : make_float4(0, 0, 0, 0);
+      }
+      for (int p = 1; p < a.planes; ++p)
+#pragma unroll
+        for (int i = 0; i < NVW; ++i) {
+          const int c = lane + i * 32;
+          if (c < nv) x[i] = fma4(1.0f, *reinterpret_cast<const float4*>(a.delta + p * a.plane + (size_t)t * a.ldx + c * 4), x[i]);
+        }
+#pragma unroll
+      for (int i = 0; i < NVW; ++i) ss += dot4(x[i]);
+      const float r = g_post / sqrtf(warp_sum(ss) * inv_w + a.eps);
+      ss = 0.0f;
+#pragma unroll
+      for (int i = 0; i < NVW; ++i) {
+        const int c = lane + i * 32;
+        if (c < nv) x[i] = fma4(r, x[i], xr[c]);
+        ss += dot4(x[i]);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < NVW; ++i) {
+        const int c = lane + i * 32;
+        x[i] = c < nv ? xr[c] : make_float4(0, 0, 0, 0);
+        ss += dot4(x[i]);
+      }
+    }
+    const float r = g_pre / sqrtf(warp_sum(ss) * inv_w + a.eps);
+    float* keep = t < r_begin ? halo + (size_t)(t - t0) * a.ldx : (a.x_out ? a.x_out + (size_t)t * a.ldx : nullptr);
+    T* out = static_cast<T*>(a.out) + (size_t)t * a.ldx;
+    if (lane == 0) s_r[t - t0] = r;
+#pragma unroll
+    for (int i = 0; i < NVW; ++i) {
+      const int c = lane + i * 32;
+      if (c >= nv) continue;
+      if (keep) store4(keep + c * 4, x[i]);
+      if (TW == 1) store4(out + c * 4, fma4(r, x[i], make_float4(0, 0, 0, 0)));
+    }
+  }
+  if (TW == 1) return;
+  __syncthreads();
+  const int keep = a.taps - 1;
+  const float* own_x = a.delta ? a.x_out : a.x_in;
+  for (int c = tid * 4; c < a.ldx; c += kNormThreads * 4) {
+    float4 w[TW], hist[TW];  // hist[s]: h of s rows ago
+#pragma unroll
+    for (int s = 0; s < TW; ++s) {
+      w[s] = s <= keep ? *reinterpret_cast<const float4*>(a.conv_w + (size_t)(keep - s) * a.ldx + c) : make_float4(0, 0, 0, 0);
+      hist[s] = make_float4(0, 0, 0, 0);
+    }
+#pragma unroll 2
+    for (int t = t0; t < r_end; ++t) {
+      const bool own = t >= r_begin;
+      const float4 x = *reinterpret_cast<const float4*>(own ? own_x + (size_t)t * a.ldx + c : halo + (size_t)(t - t0) * a.ldx + c);
+      const Entry e = a.entries[a.row_entry[t]];
+      const int off = t - e.row0;
+      const float* old_tail = a.tail + ((size_t)e.slot * 2 + e.tail) * keep * a.ldx + c;
+      float* new_tail = a.tail + ((size_t)e.slot * 2 + (e.tail ^ 1)) * keep * a.ldx + c;
+      if (off == 0) {  // a sequence's share starts: the rows before it come from its tail, or are zero
+#pragma unroll
+        for (int s = 1; s < TW; ++s)
+          hist[s] = s <= keep && s <= e.pos0 ? *reinterpret_cast<const float4*>(old_tail + (size_t)(keep - s) * a.ldx) : make_float4(0, 0, 0, 0);
+      }
+      hist[0] = fma4(s_r[t - t0], x, make_float4(0, 0, 0, 0));
+      if (own) {
+        float4 y = hist[0];
+#pragma unroll
+        for (int s = 0; s < TW; ++s)
+          y = make_float4(fmaf(w[s].x, hist[s].x, y.x), fmaf(w[s].y, hist[s].y, y.y), fmaf(w[s].z, hist[s].z, y.z), fmaf(w[s].w, hist[s].w, y.w));
+        store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c, y);
+        const int at = keep - (e.count - off);
+        if (at >= 0) store4(new_tail + (size_t)at * a.ldx, hist[0]);
+        if (off == e.count - 1)  // a short step: older rows move down
+          for (int j = 0; j + e.count < keep; ++j)
+            store4(new_tail + (size_t)j * a.ldx, *reinterpret_cast<const float4*>(old_tail + (size_t)(j + e.count) * a.ldx));
+      }
+#pragma unroll
+      for (int s = TW - 1; s > 0; --s) hist[s] = hist[s - 1];
+    }
+  }
+}
+
+template <class T, int NVW>
+cudaError_t launch_norm_rows(cudaStream_t s, const NormArgs& a) {
+  const dim3 grid((a.rows + kManyRows - 1) / kManyRows);
+  if (a.taps == 0) return launch_pdl(lm_norm_rows_kernel<T, NVW, 1>, grid, dim3(kNormThreads), 0, s, a);
+  const size_t smem = (size_t)(a.taps - 1) * a.ldx * sizeof(float);
+  if (smem > 48 * 1024) {
+    const cudaError_t r = cudaFuncSetAttribute(lm_norm_rows_kernel<T, NVW, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (r != cudaSuccess) return r;
+  }
+  return launch_pdl(lm_norm_rows_kernel<T, NVW, 4>, grid, dim3(kNormThreads), smem, s, a);
+}
+
 template <class T, int NV>
 cudaError_t launch_norm_nv(cudaStream_t s, const NormArgs& a) {
   const size_t smem = (size_t)a.taps * a.ldx * sizeof(float);
@@ -141,6 +264,13 @@ cudaError_t launch_norm_nv(cudaStream_t s, const NormArgs& a) {
 }
 template <class T>
 cudaError_t launch_norm_t(cudaStream_t s, const NormArgs& a) {
+  // enough rows for a warp each, and a convolution (if any) that fits the register window
+  if (a.rows >= 2 * kSms && !a.gather && (a.taps == 0 || (a.taps >= 2 && a.taps <= 4)) && a.ldx <= 4096) {
+    const int w = (a.ldx / 4 + 31) / 32;
+    if (w <= 8) return launch_norm_rows<T, 8>(s, a);
+    if (w <= 16) return launch_norm_rows<T, 16>(s, a);
+    return launch_norm_rows<T, 32>(s, a);
+  }
   const int per = (a.ldx / 4 + kNormThreads - 1) / kNormThreads;
   if (per <= 1) return launch_norm_nv<T, 1>(s, a);
   if (per <= 2) return launch_norm_nv<T, 2>(s, a);
@@ -154,8 +284,20 @@ __global__ void lm_embed_kernel(const int* __restrict__ tokens, const __nv_bfloa
   pdl_launch_dependents();
   pdl_wait_prior();
   const __nv_bfloat16* src = table + (size_t)tokens[blockIdx.x] * width;
-  for (int k = threadIdx.x; k < ldx; k += blockDim.x)
-    x[(size_t)blockIdx.x * ldx + k] = k < width ? __bfloat162float(src[k]) : 0.0f;
+  float* dst = x + (size_t)blockIdx.x * ldx;
+  int k0 = 0;
+  if ((width & 7) == 0) {
+    k0 = width;
+    for (int k = threadIdx.x * 8; k < width; k += blockDim.x * 8) {
+      const uint4 p = *reinterpret_cast<const uint4*>(src + k);
+      const uint32_t w[4] = {p.x, p.y, p.z, p.w};
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+        store4(dst + k + 4 * i, make_float4(__uint_as_float(w[2 * i] << 16), __uint_as_float(w[2 * i] & 0xffff0000u),
+                                            __uint_as_float(w[2 * i + 1] << 16), __uint_as_float(w[2 * i + 1] & 0xffff0000u)));
+    }
+  }
+  for (int k = k0 + threadIdx.x; k < ldx; k += blockDim.x) dst[k] = k < width ? __bfloat162float(src[k]) : 0.0f;
 }
 
 // Rows of a decode step: one token per slot, from the slots' own state.

@@ -3,10 +3,10 @@
 // coordinates) and k is multiplied by dim^-1/2.  Everything after the projections is fp32: the rotated q and k, the
 // states, the decays (powers tabulated in double precision and rounded once) and all products.
 //   * one token per sequence: lm_ret_decode_kernel updates the state in place.
-//   * prompts and portions: chunks of kChunk tokens, cut from the portion's own start.  lm_ret_rotate_kernel rotates in
-//     place, lm_ret_chunk_kernel forms every chunk's own contribution to the state, lm_ret_scan_kernel chains them
-//     (leaving the state in front of every chunk), lm_ret_output_kernel combines the part inside the chunk with the
-//     state in front of it, and applies norm and gate.
+//   * prompts and portions: chunks of kChunk tokens, cut from the portion's own start.  lm_ret_chunk_kernel forms every
+//     chunk's own contribution to the state, lm_ret_scan_kernel chains them (leaving the state in front of every chunk),
+//     lm_ret_output_kernel combines the part inside the chunk with the state in front of it, and applies norm and gate.
+//     Both rotate as they load.
 #include <algorithm>
 
 #include "../device_common.cuh"
@@ -24,6 +24,12 @@ template <>
 __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
 
 __device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
 
@@ -113,60 +119,96 @@ __global__ void __launch_bounds__(kThreads) lm_ret_decode_kernel(RetentionArgs a
         from_f32<T>(o / sqrtf(ss / (float)a.vdim + a.eps) * silu(gr[tid]));
 }
 
-// grid rows: rotates q and k in place and scales k
-__global__ void __launch_bounds__(kThreads) lm_ret_rotate_kernel(RetentionArgs a) {
-  pdl_launch_dependents();
-  pdl_wait_prior();
-  const int row = blockIdx.x, pos = a.row_sp[row].y, half = a.rot_dims >> 1, rest = a.dim - a.rot_dims;
-  const float *cr = a.cos_t + (size_t)pos * half, *sr = a.sin_t + (size_t)pos * half;
-  const float kscale = 1.0f / sqrtf((float)a.dim);
-  float* base = a.qkvg + (size_t)row * a.ld;
-  for (int i = threadIdx.x; i < 2 * a.heads * half; i += kThreads) {
-    const int h = i / half, d = i - h * half;
-    float* x = base + (size_t)h * a.dimp;
-    const float f = h < a.heads ? 1.0f : kscale;
-    const float u = x[d], v = x[d + half], c = cr[d], s = sr[d];
-    x[d] = (u * c - v * s) * f;
-    x[d + half] = (v * c + u * s) * f;
-  }
-  for (int i = threadIdx.x; i < a.heads * rest; i += kThreads) {
-    const int h = i / rest;
-    base[(size_t)(a.heads + h) * a.dimp + a.rot_dims + (i - h * rest)] *= kscale;
-  }
+// coordinates d .. d + 3 of a rotated head (rot_dims / 2 a multiple of 4)
+__device__ __forceinline__ float4 rotated4(const float* x, int d, int rot_dims, const float* cos_r, const float* sin_r) {
+  const float4 own = *reinterpret_cast<const float4*>(x + d);
+  if (d >= rot_dims) return own;
+  const int half = rot_dims >> 1, i = d < half ? d : d - half;
+  const float4 other = *reinterpret_cast<const float4*>(x + (d < half ? d + half : i));
+  const float4 c = *reinterpret_cast<const float4*>(cos_r + i), sn = *reinterpret_cast<const float4*>(sin_r + i);
+  const float sg = d < half ? -1.0f : 1.0f;
+  return make_float4(own.x * c.x + sg * (other.x * sn.x), own.y * c.y + sg * (other.y * sn.y), own.z * c.z + sg * (other.z * sn.z),
+                     own.w * c.w + sg * (other.w * sn.w));
 }
 
-// acc[r][c] += A[k][4 ty + r] * B[k][4 tx + 64 i + c], both from shared memory
+// the same for any rot_dims; coordinates past dim are the padding (zero)
+__device__ __forceinline__ float4 rotated_any(const float* x, int d, const RetentionArgs& a, int pos) {
+  const int half = a.rot_dims >> 1;
+  const float *cr = a.cos_t + (size_t)pos * half, *sr = a.sin_t + (size_t)pos * half;
+  if ((a.rot_dims & 7) == 0) return rotated4(x, d, a.rot_dims, cr, sr);
+  return make_float4(rotated(x, d, a.rot_dims, cr, sr), rotated(x, d + 1, a.rot_dims, cr, sr), rotated(x, d + 2, a.rot_dims, cr, sr),
+                     rotated(x, d + 3, a.rot_dims, cr, sr));
+}
+
+// Two fp32 products and sums per instruction.
+__device__ __forceinline__ void fma2(uint64_t& acc, uint64_t a, uint64_t b) {
+  asm("fma.rn.f32x2 %0, %1, %2, %0;" : "+l"(acc) : "l"(a), "l"(b));
+}
+__device__ __forceinline__ uint64_t both(float v) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %1};" : "=l"(r) : "f"(v));
+  return r;
+}
+__device__ __forceinline__ float2 halves(uint64_t v) {
+  float2 r;
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+  return r;
+}
+
+// A 4 x (4 NC) tile per thread: rows 4 ty .. + 3, columns 4 tx + 64 i .. + 3, two columns per accumulator.
 template <int NC>
-__device__ __forceinline__ void tile_fma(float (&acc)[4][4 * NC], const float* A, int lda, const float* B, int ldb, int n, int ty, int tx,
-                                         int cols) {
+struct Tile {
+  uint64_t v[4][2 * NC];
+  __device__ __forceinline__ void clear() {
+#pragma unroll
+    for (int r = 0; r < 4; ++r)
+#pragma unroll
+      for (int i = 0; i < 2 * NC; ++i) v[r][i] = 0;
+  }
+  // += sum over k of A[k][row] * B[k][column], both in shared memory
+  __device__ __forceinline__ void fma(const float* A, int lda, const float* B, int ldb, int n, int ty, int tx, int cols) {
+    A += ty * 4;
+    B += tx * 4;
 #pragma unroll 4
-  for (int k = 0; k < n; ++k) {
-    const float4 av = *reinterpret_cast<const float4*>(A + (size_t)k * lda + ty * 4);
-    const float ar[4] = {av.x, av.y, av.z, av.w};
+    for (int k = 0; k < n; ++k, A += lda, B += ldb) {
+      const float4 av = *reinterpret_cast<const float4*>(A);
+      const uint64_t ar[4] = {both(av.x), both(av.y), both(av.z), both(av.w)};
 #pragma unroll
-    for (int i = 0; i < NC; ++i) {
-      const int c = tx * 4 + i * 64;
-      if (c < cols) {
-        const float4 b = *reinterpret_cast<const float4*>(B + (size_t)k * ldb + c);
+      for (int i = 0; i < NC; ++i)
+        if (tx * 4 + i * 64 < cols) {
+          const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(B + i * 64);
 #pragma unroll
-        for (int r = 0; r < 4; ++r) {
-          acc[r][4 * i] = fmaf(ar[r], b.x, acc[r][4 * i]);
-          acc[r][4 * i + 1] = fmaf(ar[r], b.y, acc[r][4 * i + 1]);
-          acc[r][4 * i + 2] = fmaf(ar[r], b.z, acc[r][4 * i + 2]);
-          acc[r][4 * i + 3] = fmaf(ar[r], b.w, acc[r][4 * i + 3]);
+          for (int r = 0; r < 4; ++r) {
+            fma2(v[r][2 * i], ar[r], b.x);
+            fma2(v[r][2 * i + 1], ar[r], b.y);
+          }
         }
-      }
     }
   }
+  __device__ __forceinline__ void scale_row(int r, float f) {
+#pragma unroll
+    for (int i = 0; i < 2 * NC; ++i) {
+      const float2 h = halves(v[r][i]);
+      asm("mov.b64 %0, {%1, %2};" : "=l"(v[r][i]) : "f"(h.x * f), "f"(h.y * f));
+    }
+  }
+  __device__ __forceinline__ float4 get(int r, int i) const {
+    const float2 a = halves(v[r][2 * i]), b = halves(v[r][2 * i + 1]);
+    return make_float4(a.x, a.y, b.x, b.y);
+  }
+};
+
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
 }
 
 struct ChunkPos {
-  int row0, len;
+  int row0, len, pos;  // first row, tokens, position of the first token
 };
 __device__ __forceinline__ ChunkPos chunk_pos(const RetentionArgs& a, int chunk) {
   const int2 c = a.chunks[chunk];
   const Entry e = a.entries[c.x];
-  return {e.row0 + c.y, min(kChunk, e.count - c.y)};
+  return {e.row0 + c.y, min(kChunk, e.count - c.y), e.pos0 + c.y};
 }
 
 // grid (chunks, heads, blocks of 64 state rows): sum over the chunk of decay^(len-1-j) k_j v_j^T
@@ -182,11 +224,12 @@ __global__ void __launch_bounds__(kThreads) lm_ret_chunk_kernel(RetentionArgs a)
   const float* kb = a.qkvg + (size_t)p.row0 * a.ld + (a.heads + h) * a.dimp;
   const float* vb = a.qkvg + (size_t)p.row0 * a.ld + 2 * a.heads * a.dimp + h * a.vdimp;
   const int nd = min(64, a.dimp - d0), v4 = a.vdimp / 4;
+  const float kscale = 1.0f / sqrtf((float)a.dim);
   for (int i = tid; i < p.len * 16; i += kThreads) {
     const int j = i >> 4, c = (i & 15) * 4;
     float4 k = make_float4(0, 0, 0, 0);
-    if (c < nd) k = *reinterpret_cast<const float4*>(kb + (size_t)j * a.ld + d0 + c);
-    const float f = pw[p.len - 1 - j];
+    if (c < nd) k = rotated_any(kb + (size_t)j * a.ld, d0 + c, a, p.pos + j);
+    const float f = pw[p.len - 1 - j] * kscale;
     *reinterpret_cast<float4*>(sK + j * 64 + c) = make_float4(k.x * f, k.y * f, k.z * f, k.w * f);
   }
   for (int i = tid; i < p.len * v4; i += kThreads) {
@@ -194,8 +237,9 @@ __global__ void __launch_bounds__(kThreads) lm_ret_chunk_kernel(RetentionArgs a)
     *reinterpret_cast<float4*>(sV + j * a.vdimp + c) = *reinterpret_cast<const float4*>(vb + (size_t)j * a.ld + c);
   }
   __syncthreads();
-  float acc[4][4 * NC] = {};
-  tile_fma<NC>(acc, sK, 64, sV, a.vdimp, p.len, ty, tx, a.vdimp);
+  Tile<NC> acc;
+  acc.clear();
+  acc.fma(sK, 64, sV, a.vdimp, p.len, ty, tx, a.vdimp);
   float* dst = a.chunk_state + ((size_t)chunk * a.heads + h) * a.dimp * a.vdimp;
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
@@ -204,8 +248,7 @@ __global__ void __launch_bounds__(kThreads) lm_ret_chunk_kernel(RetentionArgs a)
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
       const int c = tx * 4 + i * 64;
-      if (c < a.vdimp)
-        *reinterpret_cast<float4*>(dst + (size_t)d * a.vdimp + c) = make_float4(acc[r][4 * i], acc[r][4 * i + 1], acc[r][4 * i + 2], acc[r][4 * i + 3]);
+      if (c < a.vdimp) *reinterpret_cast<float4*>(dst + (size_t)d * a.vdimp + c) = acc.get(r, i);
     }
   }
 }
@@ -240,19 +283,19 @@ __global__ void __launch_bounds__(kThreads) lm_ret_scan_kernel(RetentionArgs a) 
 }
 
 size_t output_smem(const RetentionArgs& a) {
-  const size_t shared_part = std::max((size_t)a.dimp * kPad, (size_t)kChunk * kPad + (size_t)kStateRows * a.vdimp);
+  const size_t shared_part = std::max((size_t)a.dimp * kPad, (size_t)kChunk * kPad + (size_t)2 * kStateRows * a.vdimp);
   return ((size_t)a.dimp * kPad + shared_part + (size_t)kChunk * a.vdimp) * 4;
 }
 
 // grid (chunks, heads)
 template <class T, int NC>
-__global__ void __launch_bounds__(kThreads) lm_ret_output_kernel(RetentionArgs a) {
+__global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kernel(RetentionArgs a) {
   extern __shared__ __align__(16) float out_smem[];
   float* sQ = out_smem;                        // [dimp][kPad]: q transposed
   float* sV = sQ + (size_t)a.dimp * kPad;      // [kChunk][vdimp]
   float* sK = sV + (size_t)kChunk * a.vdimp;   // [dimp][kPad]: k transposed; afterwards
   float* sA = sK;                              //   [kChunk][kPad]: decayed scores, transposed
-  float* sS = sA + (size_t)kChunk * kPad;      //   [kStateRows][vdimp]: rows of the state
+  float* sS = sA + (size_t)kChunk * kPad;      //   [2][kStateRows][vdimp]: rows of the state
   pdl_launch_dependents();
   pdl_wait_prior();
   const int chunk = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
@@ -263,56 +306,72 @@ __global__ void __launch_bounds__(kThreads) lm_ret_output_kernel(RetentionArgs a
   const float* vb = a.qkvg + (size_t)p.row0 * a.ld + 2 * a.heads * a.dimp + h * a.vdimp;
   const float* gb = vb + a.heads * a.vdimp;
   const int d4 = a.dimp / 4, v4 = a.vdimp / 4;
-  for (int i = tid; i < kChunk * d4; i += kThreads) {
-    const int j = i / d4, d = (i - j * d4) * 4;
+  const float kscale = 1.0f / sqrtf((float)a.dim);
+  for (int i = tid; i < p.len * v4; i += kThreads) {
+    const int j = i / v4, c = (i - j * v4) * 4;
+    cp_async16(sV + j * a.vdimp + c, vb + (size_t)j * a.ld + c);
+  }
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  for (int i = tid; i < kChunk * d4; i += kThreads) {  // lanes over tokens: the transposed stores hit 32 banks
+    const int j = i & (kChunk - 1), d = (i / kChunk) * 4;
     float4 q = make_float4(0, 0, 0, 0), k = q;
     if (j < p.len) {
-      q = *reinterpret_cast<const float4*>(qb + (size_t)j * a.ld + d);
-      k = *reinterpret_cast<const float4*>(kb + (size_t)j * a.ld + d);
+      q = rotated_any(qb + (size_t)j * a.ld, d, a, p.pos + j);
+      k = rotated_any(kb + (size_t)j * a.ld, d, a, p.pos + j);
     }
     sQ[d * kPad + j] = q.x, sQ[(d + 1) * kPad + j] = q.y, sQ[(d + 2) * kPad + j] = q.z, sQ[(d + 3) * kPad + j] = q.w;
-    sK[d * kPad + j] = k.x, sK[(d + 1) * kPad + j] = k.y, sK[(d + 2) * kPad + j] = k.z, sK[(d + 3) * kPad + j] = k.w;
-  }
-  for (int i = tid; i < kChunk * v4; i += kThreads) {
-    const int j = i / v4, c = (i - j * v4) * 4;
-    *reinterpret_cast<float4*>(sV + j * a.vdimp + c) =
-        j < p.len ? *reinterpret_cast<const float4*>(vb + (size_t)j * a.ld + c) : make_float4(0, 0, 0, 0);
+    sK[d * kPad + j] = k.x * kscale, sK[(d + 1) * kPad + j] = k.y * kscale, sK[(d + 2) * kPad + j] = k.z * kscale, sK[(d + 3) * kPad + j] = k.w * kscale;
   }
   __syncthreads();
-  {
-    float s[4][4] = {};
-    tile_fma<1>(s, sQ, kPad, sK, kPad, a.dimp, ty, tx, 64);
-    __syncthreads();  // k is no longer needed
-#pragma unroll
-    for (int c = 0; c < 4; ++c)
-#pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const int i = ty * 4 + r, j = tx * 4 + c;
-        sA[j * kPad + i] = j <= i ? s[r][c] * pw[i - j] : 0.0f;
-      }
-  }
-  float acc[4][4 * NC] = {};
   const float* S = a.chunk_state + ((size_t)chunk * a.heads + h) * a.dimp * a.vdimp;
-  for (int d0 = 0; d0 < a.dimp; d0 += kStateRows) {  // dimp is a multiple of 16
-    for (int i = tid; i < kStateRows * v4; i += kThreads)
-      reinterpret_cast<float4*>(sS)[i] = reinterpret_cast<const float4*>(S + (size_t)d0 * a.vdimp)[i];
+  auto fetch = [&](int d0) {  // kStateRows rows of the state; dimp is a multiple of them
+    float* dst = sS + (size_t)((d0 / kStateRows) & 1) * kStateRows * a.vdimp;
+    for (int i = tid; i < kStateRows * v4; i += kThreads) cp_async16(dst + 4 * i, S + (size_t)d0 * a.vdimp + 4 * i);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  {
+    Tile<1> s;
+    s.clear();
+    s.fma(sQ, kPad, sK, kPad, a.dimp, ty, tx, 64);
+    __syncthreads();  // k is no longer needed
+    fetch(0);
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+      const float4 v = s.get(r, 0);
+      const float sv[4] = {v.x, v.y, v.z, v.w};
+      const int i = ty * 4 + r;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int j = tx * 4 + c;
+        sA[j * kPad + i] = j <= i ? sv[c] * pw[i - j] : 0.0f;
+      }
+    }
+  }
+  Tile<NC> acc;
+  acc.clear();
+  for (int d0 = 0; d0 < a.dimp; d0 += kStateRows) {
+    if (d0 + kStateRows < a.dimp) {
+      fetch(d0 + kStateRows);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
     __syncthreads();
-    tile_fma<NC>(acc, sQ + (size_t)d0 * kPad, kPad, sS, a.vdimp, kStateRows, ty, tx, a.vdimp);
+    acc.fma(sQ + (size_t)d0 * kPad, kPad, sS + (size_t)((d0 / kStateRows) & 1) * kStateRows * a.vdimp, a.vdimp, kStateRows, ty, tx, a.vdimp);
     __syncthreads();
   }
 #pragma unroll
-  for (int r = 0; r < 4; ++r) {
-    const float f = pw[ty * 4 + r + 1];
-#pragma unroll
-    for (int i = 0; i < 4 * NC; ++i) acc[r][i] *= f;
-  }
-  tile_fma<NC>(acc, sA, kPad, sV, a.vdimp, min(p.len, ty / 2 * 8 + 8), ty, tx, a.vdimp);
+  for (int r = 0; r < 4; ++r) acc.scale_row(r, pw[ty * 4 + r + 1]);
+  acc.fma(sA, kPad, sV, a.vdimp, min(p.len, ty / 2 * 8 + 8), ty, tx, a.vdimp);
   T* out = static_cast<T*>(a.out);
 #pragma unroll
   for (int r = 0; r < 4; ++r) {
     float ss = 0.0f;
 #pragma unroll
-    for (int i = 0; i < 4 * NC; ++i) ss += acc[r][i] * acc[r][i];
+    for (int i = 0; i < NC; ++i) {
+      const float4 v = acc.get(r, i);
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
     const int j = ty * 4 + r;
@@ -322,12 +381,9 @@ __global__ void __launch_bounds__(kThreads) lm_ret_output_kernel(RetentionArgs a
     for (int i = 0; i < NC; ++i) {
       const int c = tx * 4 + i * 64;
       if (c < a.vdimp) {
-        const float4 g = *reinterpret_cast<const float4*>(gb + (size_t)j * a.ld + c);
-        T* o = out + (size_t)(p.row0 + j) * a.ldo + h * a.vdimp + c;
-        o[0] = from_f32<T>(acc[r][4 * i] * inv * silu(g.x));
-        o[1] = from_f32<T>(acc[r][4 * i + 1] * inv * silu(g.y));
-        o[2] = from_f32<T>(acc[r][4 * i + 2] * inv * silu(g.z));
-        o[3] = from_f32<T>(acc[r][4 * i + 3] * inv * silu(g.w));
+        const float4 g = *reinterpret_cast<const float4*>(gb + (size_t)j * a.ld + c), v = acc.get(r, i);
+        store4(out + (size_t)(p.row0 + j) * a.ldo + h * a.vdimp + c,
+               make_float4(v.x * inv * silu(g.x), v.y * inv * silu(g.y), v.z * inv * silu(g.z), v.w * inv * silu(g.w)));
       }
     }
   }
@@ -335,9 +391,7 @@ __global__ void __launch_bounds__(kThreads) lm_ret_output_kernel(RetentionArgs a
 
 template <class T, int NC>
 cudaError_t prefill_nc(cudaStream_t s, const RetentionArgs& a) {
-  cudaError_t r = launch_pdl(lm_ret_rotate_kernel, dim3(a.rows), dim3(kThreads), 0, s, a);
-  if (r == cudaSuccess)
-    r = launch_pdl(lm_ret_chunk_kernel<NC>, dim3(a.n_chunks, a.heads, (a.dimp + 63) / 64), dim3(kThreads), (size_t)kChunk * (64 + a.vdimp) * 4, s, a);
+  cudaError_t r = launch_pdl(lm_ret_chunk_kernel<NC>, dim3(a.n_chunks, a.heads, (a.dimp + 63) / 64), dim3(kThreads), (size_t)kChunk * (64 + a.vdimp) * 4, s, a);
   if (r == cudaSuccess) {
     const int n4 = a.dimp * a.vdimp / 4;
     r = launch_pdl(lm_ret_scan_kernel, dim3((n4 + kThreads - 1) / kThreads, a.heads, a.n_entries), dim3(kThreads), 0, s, a);

@@ -17,7 +17,6 @@ namespace lm {
 constexpr int kSms = 148;
 constexpr int kChunk = 64;      // tokens per retention chunk
 constexpr int kMaxSplits = 8;   // K splits of a linear whose consumer adds the partial sums
-constexpr int kDecodeKeys = 256;  // cache positions per CTA of the decode attention
 
 inline int pad_to(int v, int a) { return (v + a - 1) / a * a; }
 
@@ -121,12 +120,13 @@ cudaError_t launch_decode_prep(cudaStream_t s, int n, const int* slots, const in
 cudaError_t launch_argmax(cudaStream_t s, const float* logits, int rows, int vocab, int blocks, float2* best);
 cudaError_t launch_attention(cudaStream_t s, bool f32, const AttnShape& a, const void* q, int ldq, const int2* row_sp, int rows,
                              const void* kc, const void* vc, const float* bias, void* out, int ldo, const int4* tiles, int n_tiles,
-                             const int* single_rows, int n_single, int splits, float* part_o, float2* part_ml);
+                             const int* single_rows, int n_single, int chunk, int splits, float* part_o, float2* part_ml);
 int attention_tile_rows();
+constexpr int kMinDecodeChunk = 64;  // cache positions per CTA of the decode attention: 64, or 128 in large batches
 cudaError_t attention_configure();
 cudaError_t launch_rope_table(cudaStream_t s, float* cos_t, float* sin_t, int max_pos, int dims, double base);
 struct RetentionArgs {
-  float* qkvg;  // [rows][ld]: q | k | v | g, heads x dimp, heads x dimp, heads x vdimp, heads x vdimp
+  const float* qkvg;  // [rows][ld]: q | k | v | g, heads x dimp, heads x dimp, heads x vdimp, heads x vdimp
   int ld, heads, dim, dimp, vdim, vdimp, rot_dims;
   const float *cos_t, *sin_t, *decay;
   float* state;        // [slot][heads][dimp][vdimp]

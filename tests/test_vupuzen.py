@@ -30,7 +30,7 @@ def row_error(got, want):
 class Case:
     """A model on the GPU and in the oracle."""
 
-    def __init__(self, folder, cfg, w, dtype, max_seqs=4, max_ctx=1024, max_rows=1024):
+    def __init__(self, folder, cfg, w, dtype, max_seqs=6, max_ctx=1024, max_rows=1024):
         self.cfg, self.w, self.dtype = cfg, w, dtype
         self.model, runtime = registry.load(M.write(folder, cfg, w), dtype, max_seqs, max_ctx, max_rows)
         assert runtime == "engine"
@@ -258,9 +258,9 @@ def test_mechanism_alone(name, dtype, tmp_path):
 @pytest.mark.parametrize("name", list(M.MODELS))
 def test_prompt_and_portions(cases, name, dtype):
     c = cases(name, dtype)
-    toks = c.tokens(261)
+    toks = c.tokens(333)
     want = c.oracle(toks)
-    for portions in (None, [64], [2], [37, 2, 3, 65, 1, 1, 2, 130], [128, 1], [1, 63, 65, 7, 3]):
+    for portions in (None, [64], [2], [37, 2, 3, 65, 1, 1, 2, 130], [128, 1], [1, 63, 65, 7, 3], [5, 300]):
         c.check(c.run(toks, portions), want)
 
 
@@ -303,6 +303,28 @@ def test_mixed_batches_equal_requests_alone(cases, name, dtype):
                 m.release(live.pop(i)[0])
     for g, w in zip(got, want):
         c.check(np.concatenate(g), w)
+
+
+@gpu
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("name", list(M.MODELS))
+def test_large_ragged_steps(cases, name, dtype):
+    """Steps of several hundred rows in which sequences of one, two and hundreds of tokens meet anywhere."""
+    c = cases(name, dtype)
+    m = c.model
+    sizes = [(1, 2, 310, 1, 40, 3), (2, 1, 5, 290, 1, 17), (150, 150, 1, 3, 2, 2)]
+    reqs = [c.tokens(sum(s[i] for s in sizes), 60 + i) for i in range(6)]
+    want = [c.oracle(t) for t in reqs]
+    slots, at, got = [m.acquire() for _ in reqs], [0] * 6, [[] for _ in reqs]
+    for s in sizes:
+        logits, row = m.step([(slots[i], reqs[i][at[i]:at[i] + s[i]]) for i in range(6)], list(range(sum(s)))), 0
+        for i in range(6):
+            got[i].append(logits[row:row + s[i]])
+            row, at[i] = row + s[i], at[i] + s[i]
+    for i in range(6):
+        m.release(slots[i])
+        c.check(np.concatenate(got[i]), want[i])
+    m.check_device_status()
 
 
 @gpu
