@@ -177,6 +177,9 @@ def once(torch, mb, bench, which, size, layers):
             m.step([(x, rng.integers(0, 8192, 1024).tolist()) for x in slots[k:k + 16]], sample=True)
         m.decode(slots, 1)
         m.decode(slots[:1], 1)
+        for n, x in zip((128, 512), slots):
+            m.release(x)
+            m.step([(m.acquire(), rng.integers(0, 8192, n).tolist())], sample=True)
         m.synchronize()
         m.check_device_status()
         m.close()

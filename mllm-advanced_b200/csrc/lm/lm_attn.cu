@@ -4,7 +4,7 @@
 // the caches already.  Scores, weights and sums are fp32; the bf16 kernels multiply bf16 queries and keys exactly into
 // fp32 and feed the weights to the value product as a sum of two bf16 numbers.
 //   * lm_attn_prefill_kernel: tiles of 64 (token, head) rows that share a kv head, key blocks of 64 through a
-//     double-buffered cp.async ring, mma.sync m16n8k16, online softmax in registers.
+//     double-buffered cp.async ring, mma.sync m16n8k16, online softmax in registers, two warps per 16 rows.
 //   * lm_attn_decode_kernel + lm_attn_combine_kernel: one token per sequence, the context split over CTAs in chunks of 64
 //     or 128 positions, the query heads of a kv head as the rows of one mma tile.
 //   * lm_attn_f32_kernel: the 32-bit mode, any step.
@@ -85,7 +85,7 @@ __global__ void __launch_bounds__(kF32Threads) lm_attn_f32_kernel(AttnShape a, c
 }
 
 // ------------------------------------------------------------------------------------------ bf16 prompts
-constexpr int kPfRows = 64, kPfKeys = 64, kPfThreads = 128;
+constexpr int kPfRows = 64, kPfKeys = 64, kPfThreads = 256;
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
@@ -112,13 +112,24 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-size_t prefill_smem(const AttnShape& a) {
-  const int group = a.heads / a.kv_heads, toks = kPfRows / group;
-  return (size_t)(3 * kPfKeys) * (a.dimp + 8) * 2 + (size_t)(2 * kPfKeys) * (a.vdimp + 8) * 2 +
-         (a.has_bias ? (size_t)2 * group * (kPfKeys + toks) * 4 : 0);
+__device__ __forceinline__ float fast_exp2(float x) {  // results below 2^-126 are 0
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 
-// grid (tiles, kv heads); tile = {first row, tokens, slot, position of the first token}
+// entries of a tile's bias window per head: distances of all (token, key) pairs, rounded up to whole 16-byte pieces
+__host__ __device__ inline int bias_window(int toks) { return (kPfKeys + toks + 3) / 4 * 4; }
+
+size_t prefill_smem(const AttnShape& a) {
+  const int group = a.heads / a.kv_heads, toks = kPfRows / group;
+  const size_t kv = (size_t)(2 * kPfKeys) * (a.dimp + 8) * 2 + (size_t)(2 * kPfKeys) * (a.vdimp + 8) * 2;
+  return (size_t)kPfRows * (a.dimp + 8) * 2 + std::max(kv, (size_t)kPfRows * a.vdimp * 4) +
+         (a.has_bias ? (size_t)2 * group * bias_window(toks) * 4 : 0);
+}
+
+// grid (tiles, kv heads); tile = {first row, tokens, slot, position of the first token}.  Eight warps: warp w and warp
+// w + 4 own the same 16 rows and one half each of every key block; their online-softmax states meet at the end.
 template <int DV>
 __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, int ldq,
                                                                      const __nv_bfloat16* __restrict__ kc,
@@ -126,59 +137,68 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
                                                                      const float* __restrict__ bias, const int4* __restrict__ tiles,
                                                                      __nv_bfloat16* __restrict__ out, int ldo) {
   extern __shared__ __align__(16) uint8_t pf_smem[];
+  __shared__ float s_m[kPfRows], s_l[kPfRows];
+  constexpr int kHalf = kPfKeys / 2;
   const int D = a.dimp, group = a.heads / a.kv_heads, toks = kPfRows / group;
-  const int ldk = D + 8, ldv = a.vdimp + 8, win = kPfKeys + toks;
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(pf_smem);
+  const int ldk = D + 8, ldv = a.vdimp + 8, win = bias_window(toks);
+  // [2][group][win] biases | queries | 2 x keys | 2 x values; the partial outputs of warps 4..7 overlay keys and values
+  float* sB = reinterpret_cast<float*>(pf_smem);
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(sB + (a.has_bias ? 2 * group * win : 0));
   __nv_bfloat16* sK = sQ + kPfRows * ldk;
   __nv_bfloat16* sV = sK + 2 * kPfKeys * ldk;
-  float* sB = reinterpret_cast<float*>(sV + 2 * kPfKeys * ldv);  // [2][group][win]
+  float* sO = reinterpret_cast<float*>(sK);
   pdl_launch_dependents();
   pdl_wait_prior();
   const int4 tile = tiles[blockIdx.x];
-  const int kvh = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int kvh = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = warp >> 2, wrow = (warp & 3) * 16;
   const int row0 = tile.x, ntok = tile.y, pos0 = tile.w, last = pos0 + ntok - 1;
   const __nv_bfloat16* kb = kc + ((size_t)tile.z * a.kv_heads + kvh) * a.max_ctx * D;
   const __nv_bfloat16* vb = vc + ((size_t)tile.z * a.kv_heads + kvh) * a.max_ctx * a.vdimp;
   const int dv8 = D / 8, vv8 = a.vdimp / 8;
-  for (int i = tid; i < kPfRows * dv8; i += kPfThreads) {
-    const int r = i / dv8, c = i - r * dv8, tok = r / group, hg = r - tok * group;
+  // copies: eight threads per row of 16-byte pieces
+  const int cr = tid >> 3, cc = tid & 7;
+  for (int r = cr; r < kPfRows; r += kPfThreads / 8) {
+    const int tok = r / group, hg = r - tok * group;
     const bool ok = tok < ntok && tok < toks;
-    cp_async16(smem_u32(sQ + r * ldk + c * 8), q + (size_t)(row0 + (ok ? tok : 0)) * ldq + (kvh * group + hg) * D + c * 8, ok);
+    const __nv_bfloat16* src = q + (size_t)(row0 + (ok ? tok : 0)) * ldq + (kvh * group + hg) * D;
+    for (int c = cc; c < dv8; c += 8) cp_async16(smem_u32(sQ + r * ldk + c * 8), src + c * 8, ok);
   }
   auto fetch = [&](int j0, int buf) {
-    for (int i = tid; i < kPfKeys * dv8; i += kPfThreads) {
-      const int r = i / dv8, c = i - r * dv8;
+#pragma unroll
+    for (int u = 0; u < kPfKeys / (kPfThreads / 8); ++u) {
+      const int r = cr + u * (kPfThreads / 8);
       const bool ok = j0 + r <= last;
-      cp_async16(smem_u32(sK + (buf * kPfKeys + r) * ldk + c * 8), kb + (size_t)(ok ? j0 + r : 0) * D + c * 8, ok);
-    }
-    for (int i = tid; i < kPfKeys * vv8; i += kPfThreads) {
-      const int r = i / vv8, c = i - r * vv8;
-      const bool ok = j0 + r <= last;
-      cp_async16(smem_u32(sV + (buf * kPfKeys + r) * ldv + c * 8), vb + (size_t)(ok ? j0 + r : 0) * a.vdimp + c * 8, ok);
+      const size_t at = ok ? j0 + r : 0;
+      const uint32_t dk = smem_u32(sK + (buf * kPfKeys + r) * ldk), dv = smem_u32(sV + (buf * kPfKeys + r) * ldv);
+      for (int c = cc; c < dv8; c += 8) cp_async16(dk + c * 16, kb + at * D + c * 8, ok);
+      for (int c = cc; c < vv8; c += 8) cp_async16(dv + c * 16, vb + at * a.vdimp + c * 8, ok);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   fetch(0, 0);
-  // this thread's two rows of the tile
-  int tok_r[2], hg_r[2];
+  // this thread's two rows of the tile (rows past the tile's tokens compute on zeros and are not stored)
+  int tok_r[2], hg_r[2], b_at[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
-    const int r = warp * 16 + (lane >> 2) + i * 8;
+    const int r = wrow + (lane >> 2) + i * 8;
     tok_r[i] = r / group;
     hg_r[i] = r - tok_r[i] * group;
+    b_at[i] = hg_r[i] * win + min(tok_r[i], toks - 1) + kPfKeys - 1 - half * kHalf - (lane & 3) * 2;
   }
+  // the mask value is far below every running maximum, so that masked weights come out as 0
+  constexpr float kStart = -1e30f;
   float m[2], l[2], o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
-    m[i] = a.sink ? 0.0f : kNegInf;
-    l[i] = a.sink && (lane & 3) == 0 ? 1.0f : 0.0f;
+    m[i] = a.sink ? 0.0f : kStart;
+    l[i] = a.sink && half == 0 && (lane & 3) == 0 ? 1.0f : 0.0f;
   }
 #pragma unroll
   for (int n = 0; n < DV / 8; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
   const int mat = lane >> 3, ml = lane & 7;
-  const uint32_t q_addr = smem_u32(sQ + (warp * 16 + (mat & 1) * 8 + ml) * ldk + (mat >> 1) * 8);
-  const uint32_t k_addr = smem_u32(sK + ((mat >> 1) * 8 + ml) * ldk + (mat & 1) * 8);
-  const uint32_t v_addr = smem_u32(sV + ((mat & 1) * 8 + ml) * ldv + (mat >> 1) * 8);
+  const uint32_t q_addr = smem_u32(sQ + (wrow + (mat & 1) * 8 + ml) * ldk + (mat >> 1) * 8);
+  const uint32_t k_addr = smem_u32(sK + (half * kHalf + (mat >> 1) * 8 + ml) * ldk + (mat & 1) * 8);
+  const uint32_t v_addr = smem_u32(sV + (half * kHalf + (mat & 1) * 8 + ml) * ldv + (mat >> 1) * 8);
   const float sc2 = a.scale * kLog2e;
 
   for (int j0 = 0, blk = 0; j0 <= last; j0 += kPfKeys, ++blk) {
@@ -186,21 +206,23 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
     float* bw = sB + (size_t)buf * group * win;
     const int n_lo = pos0 - (j0 + kPfKeys - 1);  // distance of the window's first entry
     if (a.has_bias)
-      for (int i = tid; i < group * win; i += kPfThreads) {
-        const int hg = i / win, n = n_lo + (i - hg * win);
-        bw[i] = kLog2e * __ldg(bias + (size_t)(kvh * group + hg) * (a.bias_max + 1) + min(max(n, 0), a.bias_max));
+      for (int hg = warp; hg < group; hg += kPfThreads / 32) {
+        const float* bh = bias + (size_t)(kvh * group + hg) * (a.bias_max + 1);
+        for (int i = lane; i < win; i += 32) bw[hg * win + i] = kLog2e * __ldg(bh + min(max(n_lo + i, 0), a.bias_max));
       }
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     if (j0 + kPfKeys <= last) fetch(j0 + kPfKeys, buf ^ 1);
-    float s[kPfKeys / 8][4];
+    const int jw = j0 + half * kHalf;  // this warp's first key
+    float s[kHalf / 8][4];
 #pragma unroll
-    for (int n = 0; n < kPfKeys / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.0f;
+    for (int n = 0; n < kHalf / 8; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.0f;
+#pragma unroll 4
     for (int kk = 0; kk < D; kk += 16) {
       uint32_t qa[4];
       ldsm4(qa, q_addr + kk * 2);
 #pragma unroll
-      for (int n = 0; n < kPfKeys / 16; ++n) {
+      for (int n = 0; n < kHalf / 16; ++n) {
         uint32_t b[4];
         ldsm4(b, k_addr + ((buf * kPfKeys + n * 16) * ldk + kk) * 2);
         mma_bf16(s[2 * n], qa, b[0], b[1]);
@@ -209,38 +231,43 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
     }
     float mx[2] = {m[0], m[1]};
 #pragma unroll
-    for (int n = 0; n < kPfKeys / 8; ++n)
+    for (int n = 0; n < kHalf / 8; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int r = i >> 1, c = n * 8 + (lane & 3) * 2 + (i & 1);
-        const int dist = pos0 + tok_r[r] - (j0 + c);
-        float v = s[n][i] * sc2;
-        if (a.has_bias) v += bw[hg_r[r] * win + min(dist - n_lo, win - 1)];
-        v = dist >= 0 && tok_r[r] < ntok ? v : kNegInf;
-        s[n][i] = v;
-        mx[r] = fmaxf(mx[r], v);
+        const float b = a.has_bias ? bw[b_at[i >> 1] - n * 8 - (i & 1)] : 0.0f;
+        s[n][i] = fmaf(s[n][i], sc2, b);
       }
+    if (jw + kHalf - 1 > pos0) {  // some keys are later than some rows
+#pragma unroll
+      for (int n = 0; n < kHalf / 8; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if (jw + n * 8 + (lane & 3) * 2 + (i & 1) > pos0 + tok_r[i >> 1]) s[n][i] = kNegInf;
+    }
+#pragma unroll
+    for (int n = 0; n < kHalf / 8; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) mx[i >> 1] = fmaxf(mx[i >> 1], s[n][i]);
     float alpha[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
       mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
       mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-      alpha[r] = exp2f(m[r] - mx[r]);
+      alpha[r] = fast_exp2(m[r] - mx[r]);
       m[r] = mx[r];
       l[r] *= alpha[r];
     }
 #pragma unroll
-    for (int n = 0; n < kPfKeys / 8; ++n)
+    for (int n = 0; n < kHalf / 8; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float p = s[n][i] == kNegInf ? 0.0f : exp2f(s[n][i] - m[i >> 1]);
-        s[n][i] = p;
-        l[i >> 1] += p;
+        s[n][i] = fast_exp2(s[n][i] - m[i >> 1]);
+        l[i >> 1] += s[n][i];
       }
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n) o[n][0] *= alpha[0], o[n][1] *= alpha[0], o[n][2] *= alpha[1], o[n][3] *= alpha[1];
 #pragma unroll
-    for (int kk = 0; kk < kPfKeys / 16; ++kk) {
+    for (int kk = 0; kk < kHalf / 16; ++kk) {
       uint32_t hi[4], lo[4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
@@ -254,8 +281,8 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
           uint32_t b[4];
           ldsm4_t(b, v_addr + ((buf * kPfKeys + kk * 16) * ldv + n * 16) * 2);
           mma_bf16(o[2 * n], hi, b[0], b[1]);
-          mma_bf16(o[2 * n], lo, b[0], b[1]);
           mma_bf16(o[2 * n + 1], hi, b[2], b[3]);
+          mma_bf16(o[2 * n], lo, b[0], b[1]);
           mma_bf16(o[2 * n + 1], lo, b[2], b[3]);
         }
       }
@@ -265,12 +292,35 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
   for (int r = 0; r < 2; ++r) {
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
     l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
+  }
+  __syncthreads();  // keys and values are used up
+  if (half == 1) {
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int row = wrow + (lane >> 2) + r * 8;
+      if ((lane & 3) == 0) s_m[row] = m[r], s_l[row] = l[r];
+      float* so = sO + (size_t)row * a.vdimp + (lane & 3) * 2;
+#pragma unroll
+      for (int n = 0; n < DV / 8; ++n)
+        if (n * 8 < a.vdimp) *reinterpret_cast<float2*>(so + n * 8) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
+    }
+  }
+  __syncthreads();
+  if (half == 1) return;
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
     if (tok_r[r] >= ntok || tok_r[r] >= toks) continue;
-    const float inv = 1.0f / l[r];
+    const int row = wrow + (lane >> 2) + r * 8;
+    const float mo = s_m[row], mt = fmaxf(m[r], mo), f0 = fast_exp2(m[r] - mt), f1 = fast_exp2(mo - mt);
+    const float inv = 1.0f / (l[r] * f0 + s_l[row] * f1), g0 = f0 * inv, g1 = f1 * inv;
+    const float* so = sO + (size_t)row * a.vdimp + (lane & 3) * 2;
     __nv_bfloat16* orow = out + (size_t)(row0 + tok_r[r]) * ldo + (kvh * group + hg_r[r]) * a.vdimp + (lane & 3) * 2;
 #pragma unroll
     for (int n = 0; n < DV / 8; ++n)
-      if (n * 8 < a.vdimp) *reinterpret_cast<uint32_t*>(orow + n * 8) = pack2(o[n][2 * r] * inv, o[n][2 * r + 1] * inv);
+      if (n * 8 < a.vdimp) {
+        const float2 w = *reinterpret_cast<const float2*>(so + n * 8);
+        *reinterpret_cast<uint32_t*>(orow + n * 8) = pack2(fmaf(o[n][2 * r], g0, w.x * g1), fmaf(o[n][2 * r + 1], g0, w.y * g1));
+      }
   }
 }
 
@@ -313,18 +363,21 @@ __global__ void __launch_bounds__(kDecThreads) lm_attn_decode_kernel(AttnShape a
   const int nh = min(kDecRows, group - hb0), h0 = kvh * group + hb0, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const size_t base = ((size_t)sp.x * a.kv_heads + kvh) * a.max_ctx + j0;
   const int dv8 = D / 8, vv8 = a.vdimp / 8;
-  for (int i = tid; i < kDecRows * dv8; i += kDecThreads) {
-    const int r = i / dv8, c = i - r * dv8;
-    cp_async16(smem_u32(sQ + r * ldk + c * 8), q + (size_t)row * ldq + (size_t)(h0 + (r < nh ? r : 0)) * D + c * 8, r < nh);
-  }
-  for (int i = tid; i < kKeys * dv8; i += kDecThreads) {
-    const int r = i / dv8, c = i - r * dv8;
-    cp_async16(smem_u32(sK + r * ldk + c * 8), kc + (base + (r < nk ? r : 0)) * D + c * 8, r < nk);
+  const int cr = tid >> 3, cc = tid & 7;  // copies: eight threads per row of 16-byte pieces
+  for (int c = cc; c < dv8; c += 8)
+    cp_async16(smem_u32(sQ + cr * ldk + c * 8), q + (size_t)row * ldq + (size_t)(h0 + (cr < nh ? cr : 0)) * D + c * 8, cr < nh);
+#pragma unroll
+  for (int u = 0; u < kKeys / 16; ++u) {
+    const int r = cr + u * 16;
+    const __nv_bfloat16* src = kc + (base + (r < nk ? r : 0)) * D;
+    for (int c = cc; c < dv8; c += 8) cp_async16(smem_u32(sK + r * ldk + c * 8), src + c * 8, r < nk);
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
-  for (int i = tid; i < kKeys * vv8; i += kDecThreads) {
-    const int r = i / vv8, c = i - r * vv8;
-    cp_async16(smem_u32(sV + r * ldv + c * 8), vc + (base + (r < nk ? r : 0)) * a.vdimp + c * 8, r < nk);
+#pragma unroll
+  for (int u = 0; u < kKeys / 16; ++u) {
+    const int r = cr + u * 16;
+    const __nv_bfloat16* src = vc + (base + (r < nk ? r : 0)) * a.vdimp;
+    for (int c = cc; c < vv8; c += 8) cp_async16(smem_u32(sV + r * ldv + c * 8), src + c * 8, r < nk);
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
   const int k0 = warp * 16 * WK, mat = lane >> 3, ml = lane & 7;

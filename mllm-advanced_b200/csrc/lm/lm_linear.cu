@@ -450,7 +450,8 @@ void choose_tile(int M, int N, int K, int max_splits, int* bn_out, int* splits_o
       const long long items = (long long)mt * nt * s;
       const double waves = (double)((items + kSms - 1) / kSms);
       const double per_k = std::max(2.0 * bn, (a_rows + bn) * 128.0 / 40.0);
-      const double t = waves * (((kt + s - 1) / s) * per_k + 600.0 + 6.0 * bn) + 900.0 + (s - 1) * 150.0;
+      // more planes are written here and read by the consumer: about 2600 bytes per cycle
+      const double t = waves * (((kt + s - 1) / s) * per_k + 600.0 + 6.0 * bn) + 900.0 + (s - 1) * (150.0 + 8.0 * M * N / 2600.0);
       if (t < best) best = t, *bn_out = bn, *splits_out = s;
     }
   }

@@ -133,17 +133,18 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
 // The same for many rows: a warp per row for the sums (no block barrier inside), then - with a convolution - the threads
 // sweep the CTA's rows column by column with the last TW - 1 rows of h in registers.  x' of the CTA's own rows is read
 // back from x_out (or x_in when there is nothing to fold in), that of the rows in front of them from shared memory.
-constexpr int kManyRows = 16, kNormWarps = kNormThreads / 32;
+constexpr int kRowsThreads = 384, kRowsWarps = kRowsThreads / 32;  // rows a CTA handles at once, the recomputed ones included
 
 template <class T, int NVW, int TW>
-__global__ void __launch_bounds__(kNormThreads) lm_norm_rows_kernel(NormArgs a) {
+__global__ void __launch_bounds__(kRowsThreads) lm_norm_rows_kernel(NormArgs a) {
   extern __shared__ __align__(16) float halo[];  // [TW - 1][ldx]
-  __shared__ float s_r[kManyRows + 8];
+  __shared__ float s_r[2 * kRowsWarps];
+  __shared__ Entry s_e[2 * kRowsWarps];
   pdl_launch_dependents();
   pdl_wait_prior();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nv = a.ldx >> 2;
   const float g_pre = *a.g_pre, g_post = a.delta ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
-  const int r_begin = blockIdx.x * kManyRows, r_end = min(r_begin + kManyRows, a.rows);
+  const int r_begin = blockIdx.x * a.rows_per_cta, r_end = min(r_begin + a.rows_per_cta, a.rows);
   int t0 = r_begin;
   if (TW > 1) t0 = max(r_begin - (a.taps - 1), a.entries[a.row_entry[r_begin]].row0);
   auto warp_sum = [](float v) {
@@ -151,7 +152,8 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_rows_kernel(NormArgs a) 
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
   };
-  for (int t = t0 + warp; t < r_end; t += kNormWarps) {
+  if (TW > 1 && tid < r_end - t0) s_e[tid] = a.entries[a.row_entry[t0 + tid]];
+  for (int t = t0 + warp; t < r_end; t += kRowsWarps) {
     const float4* xr = reinterpret_cast<const float4*>(a.x_in + (size_t)t * a.ldx);
     float4 x[NVW];
     float ss = 0.0f;
@@ -202,55 +204,68 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_rows_kernel(NormArgs a) 
   __syncthreads();
   const int keep = a.taps - 1;
   const float* own_x = a.delta ? a.x_out : a.x_in;
-  for (int c = tid * 4; c < a.ldx; c += kNormThreads * 4) {
+  for (int c = tid * 4; c < a.ldx; c += kRowsThreads * 4) {
     float4 w[TW], hist[TW];  // hist[s]: h of s rows ago
 #pragma unroll
     for (int s = 0; s < TW; ++s) {
       w[s] = s <= keep ? *reinterpret_cast<const float4*>(a.conv_w + (size_t)(keep - s) * a.ldx + c) : make_float4(0, 0, 0, 0);
       hist[s] = make_float4(0, 0, 0, 0);
     }
-#pragma unroll 2
-    for (int t = t0; t < r_end; ++t) {
-      const bool own = t >= r_begin;
-      const float4 x = *reinterpret_cast<const float4*>(own ? own_x + (size_t)t * a.ldx + c : halo + (size_t)(t - t0) * a.ldx + c);
-      const Entry e = a.entries[a.row_entry[t]];
-      const int off = t - e.row0;
-      const float* old_tail = a.tail + ((size_t)e.slot * 2 + e.tail) * keep * a.ldx + c;
-      float* new_tail = a.tail + ((size_t)e.slot * 2 + (e.tail ^ 1)) * keep * a.ldx + c;
-      if (off == 0) {  // a sequence's share starts: the rows before it come from its tail, or are zero
+    for (int tb = t0; tb < r_end; tb += kRowsWarps) {
+      float4 x[kRowsWarps];
 #pragma unroll
-        for (int s = 1; s < TW; ++s)
-          hist[s] = s <= keep && s <= e.pos0 ? *reinterpret_cast<const float4*>(old_tail + (size_t)(keep - s) * a.ldx) : make_float4(0, 0, 0, 0);
-      }
-      hist[0] = fma4(s_r[t - t0], x, make_float4(0, 0, 0, 0));
-      if (own) {
-        float4 y = hist[0];
-#pragma unroll
-        for (int s = 0; s < TW; ++s)
-          y = make_float4(fmaf(w[s].x, hist[s].x, y.x), fmaf(w[s].y, hist[s].y, y.y), fmaf(w[s].z, hist[s].z, y.z), fmaf(w[s].w, hist[s].w, y.w));
-        store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c, y);
-        const int at = keep - (e.count - off);
-        if (at >= 0) store4(new_tail + (size_t)at * a.ldx, hist[0]);
-        if (off == e.count - 1)  // a short step: older rows move down
-          for (int j = 0; j + e.count < keep; ++j)
-            store4(new_tail + (size_t)j * a.ldx, *reinterpret_cast<const float4*>(old_tail + (size_t)(j + e.count) * a.ldx));
+      for (int u = 0; u < kRowsWarps; ++u) {
+        const int t = tb + u;
+        if (t < r_end) x[u] = *reinterpret_cast<const float4*>(t >= r_begin ? own_x + (size_t)t * a.ldx + c : halo + (size_t)(t - t0) * a.ldx + c);
       }
 #pragma unroll
-      for (int s = TW - 1; s > 0; --s) hist[s] = hist[s - 1];
+      for (int u = 0; u < kRowsWarps; ++u) {
+        const int t = tb + u;
+        if (t >= r_end) break;
+        const Entry e = s_e[t - t0];
+        const int off = t - e.row0;
+        if (off == 0) {  // a sequence's share starts: the rows before it come from its tail, or are zero
+          const float* old_tail = a.tail + ((size_t)e.slot * 2 + e.tail) * keep * a.ldx + c;
+#pragma unroll
+          for (int s = 1; s < TW; ++s)
+            hist[s] = s <= keep && s <= e.pos0 ? *reinterpret_cast<const float4*>(old_tail + (size_t)(keep - s) * a.ldx) : make_float4(0, 0, 0, 0);
+        }
+        hist[0] = fma4(s_r[t - t0], x[u], make_float4(0, 0, 0, 0));
+        if (t >= r_begin) {
+          float4 y = hist[0];
+#pragma unroll
+          for (int s = 0; s < TW; ++s)
+            y = make_float4(fmaf(w[s].x, hist[s].x, y.x), fmaf(w[s].y, hist[s].y, y.y), fmaf(w[s].z, hist[s].z, y.z), fmaf(w[s].w, hist[s].w, y.w));
+          store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c, y);
+          const int at = keep - (e.count - off);
+          if (at >= 0) {  // among the last rows of its sequence's share: the new tail
+            const float* old_tail = a.tail + ((size_t)e.slot * 2 + e.tail) * keep * a.ldx + c;
+            float* new_tail = a.tail + ((size_t)e.slot * 2 + (e.tail ^ 1)) * keep * a.ldx + c;
+            store4(new_tail + (size_t)at * a.ldx, hist[0]);
+            if (off == e.count - 1)  // a short step: older rows move down
+              for (int j = 0; j + e.count < keep; ++j)
+                store4(new_tail + (size_t)j * a.ldx, *reinterpret_cast<const float4*>(old_tail + (size_t)(j + e.count) * a.ldx));
+          }
+        }
+#pragma unroll
+        for (int s = TW - 1; s > 0; --s) hist[s] = hist[s - 1];
+      }
     }
   }
 }
 
 template <class T, int NVW>
-cudaError_t launch_norm_rows(cudaStream_t s, const NormArgs& a) {
-  const dim3 grid((a.rows + kManyRows - 1) / kManyRows);
-  if (a.taps == 0) return launch_pdl(lm_norm_rows_kernel<T, NVW, 1>, grid, dim3(kNormThreads), 0, s, a);
-  const size_t smem = (size_t)(a.taps - 1) * a.ldx * sizeof(float);
-  if (smem > 48 * 1024) {
+cudaError_t launch_norm_rows(cudaStream_t s, NormArgs a) {
+  const int halo = a.taps ? a.taps - 1 : 0;
+  a.rows_per_cta = (a.rows >= 4 * kSms * kRowsWarps ? 2 : 1) * kRowsWarps - halo;
+  const dim3 grid((a.rows + a.rows_per_cta - 1) / a.rows_per_cta);
+  if (a.taps == 0) return launch_pdl(lm_norm_rows_kernel<T, NVW, 1>, grid, dim3(kRowsThreads), 0, s, a);
+  const size_t smem = (size_t)halo * a.ldx * sizeof(float);
+  if (smem > 40 * 1024) {
     const cudaError_t r = cudaFuncSetAttribute(lm_norm_rows_kernel<T, NVW, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (r != cudaSuccess) return r;
   }
-  return launch_pdl(lm_norm_rows_kernel<T, NVW, 4>, grid, dim3(kNormThreads), smem, s, a);
+  return launch_pdl(lm_norm_rows_kernel<T, NVW, 4>, grid, dim3(kRowsThreads), smem, s, a);
 }
 
 template <class T, int NV>

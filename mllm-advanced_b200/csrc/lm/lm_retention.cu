@@ -165,24 +165,26 @@ struct Tile {
 #pragma unroll
       for (int i = 0; i < 2 * NC; ++i) v[r][i] = 0;
   }
-  // += sum over k of A[k][row] * B[k][column], both in shared memory
+  // += sum over k of A[k][row] * B[k][column], both in shared memory.  Columns past `cols` repeat column 0: they hold
+  // something, and nobody stores it.
   __device__ __forceinline__ void fma(const float* A, int lda, const float* B, int ldb, int n, int ty, int tx, int cols) {
     A += ty * 4;
-    B += tx * 4;
+    const float* b[NC];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) b[i] = B + (tx * 4 + i * 64 < cols ? tx * 4 + i * 64 : 0);
 #pragma unroll 4
-    for (int k = 0; k < n; ++k, A += lda, B += ldb) {
-      const float4 av = *reinterpret_cast<const float4*>(A);
+    for (int k = 0; k < n; ++k) {
+      const float4 av = *reinterpret_cast<const float4*>(A + k * lda);
       const uint64_t ar[4] = {both(av.x), both(av.y), both(av.z), both(av.w)};
 #pragma unroll
-      for (int i = 0; i < NC; ++i)
-        if (tx * 4 + i * 64 < cols) {
-          const ulonglong2 b = *reinterpret_cast<const ulonglong2*>(B + i * 64);
+      for (int i = 0; i < NC; ++i) {
+        const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(b[i] + k * ldb);
 #pragma unroll
-          for (int r = 0; r < 4; ++r) {
-            fma2(v[r][2 * i], ar[r], b.x);
-            fma2(v[r][2 * i + 1], ar[r], b.y);
-          }
+        for (int r = 0; r < 4; ++r) {
+          fma2(v[r][2 * i], ar[r], bv.x);
+          fma2(v[r][2 * i + 1], ar[r], bv.y);
         }
+      }
     }
   }
   __device__ __forceinline__ void scale_row(int r, float f) {
@@ -369,6 +371,7 @@ __global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kerne
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
+      if (tx * 4 + i * 64 >= a.vdimp) break;
       const float4 v = acc.get(r, i);
       ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
