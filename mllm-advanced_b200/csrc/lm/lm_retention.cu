@@ -17,6 +17,7 @@ namespace lm {
 namespace {
 
 constexpr int kThreads = 256, kPad = kChunk + 4, kStateRows = 16;
+constexpr int kRows = 8, kTileThreads = kChunk / kRows * 16;  // of the tiled products: rows per thread, threads per 64 rows
 
 template <class T>
 __device__ __forceinline__ T from_f32(float v);
@@ -155,36 +156,49 @@ __device__ __forceinline__ float2 halves(uint64_t v) {
   return r;
 }
 
-// A 4 x (4 NC) tile per thread: rows 4 ty .. + 3, columns 4 tx + 64 i .. + 3, two columns per accumulator.
+// A kRows x (4 NC) tile per thread: rows kRows ty .., columns 4 tx + 64 i .. + 3, two columns per accumulator.
 template <int NC>
 struct Tile {
-  uint64_t v[4][2 * NC];
+  uint64_t v[kRows][2 * NC];
   __device__ __forceinline__ void clear() {
 #pragma unroll
-    for (int r = 0; r < 4; ++r)
+    for (int r = 0; r < kRows; ++r)
 #pragma unroll
       for (int i = 0; i < 2 * NC; ++i) v[r][i] = 0;
   }
-  // += sum over k of A[k][row] * B[k][column], both in shared memory.  Columns past `cols` repeat column 0: they hold
-  // something, and nobody stores it.
+  // += sum over k of a(k, row) * B[k][column], in shared memory; a(k, row) = A[row][k] (KMAJOR; n a multiple of 4) or
+  // A[k][row].  Columns past `cols` repeat column 0: they hold something, and nobody stores it.
+  template <bool KMAJOR>
   __device__ __forceinline__ void fma(const float* A, int lda, const float* B, int ldb, int n, int ty, int tx, int cols) {
-    A += ty * 4;
+    constexpr int kStep = KMAJOR ? 4 : 1;
+    A += ty * kRows * (KMAJOR ? lda : 1);
     const float* b[NC];
 #pragma unroll
     for (int i = 0; i < NC; ++i) b[i] = B + (tx * 4 + i * 64 < cols ? tx * 4 + i * 64 : 0);
-#pragma unroll 4
-    for (int k = 0; k < n; ++k) {
-      const float4 av = *reinterpret_cast<const float4*>(A + k * lda);
-      const uint64_t ar[4] = {both(av.x), both(av.y), both(av.z), both(av.w)};
+#pragma unroll 2
+    for (int k0 = 0; k0 < n; k0 += kStep) {
+      float av[kRows][kStep];
+      if (KMAJOR) {
 #pragma unroll
-      for (int i = 0; i < NC; ++i) {
-        const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(b[i] + k * ldb);
+        for (int r = 0; r < kRows; ++r) *reinterpret_cast<float4*>(av[r]) = *reinterpret_cast<const float4*>(A + r * lda + k0);
+      } else {
 #pragma unroll
-        for (int r = 0; r < 4; ++r) {
-          fma2(v[r][2 * i], ar[r], bv.x);
-          fma2(v[r][2 * i + 1], ar[r], bv.y);
+        for (int r = 0; r < kRows; r += 4) {
+          const float4 t = *reinterpret_cast<const float4*>(A + k0 * lda + r);
+          av[r][0] = t.x, av[r + 1][0] = t.y, av[r + 2][0] = t.z, av[r + 3][0] = t.w;
         }
       }
+#pragma unroll
+      for (int kk = 0; kk < kStep; ++kk)
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+          const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(b[i] + (k0 + kk) * ldb);
+#pragma unroll
+          for (int r = 0; r < kRows; ++r) {
+            fma2(v[r][2 * i], both(av[r][kk]), bv.x);
+            fma2(v[r][2 * i + 1], both(av[r][kk]), bv.y);
+          }
+        }
     }
   }
   __device__ __forceinline__ void scale_row(int r, float f) {
@@ -215,7 +229,7 @@ __device__ __forceinline__ ChunkPos chunk_pos(const RetentionArgs& a, int chunk)
 
 // grid (chunks, heads, blocks of 64 state rows): sum over the chunk of decay^(len-1-j) k_j v_j^T
 template <int NC>
-__global__ void __launch_bounds__(kThreads) lm_ret_chunk_kernel(RetentionArgs a) {
+__global__ void __launch_bounds__(kTileThreads) lm_ret_chunk_kernel(RetentionArgs a) {
   extern __shared__ __align__(16) float ck_smem[];
   float *sK = ck_smem, *sV = sK + kChunk * 64;  // [kChunk][64], [kChunk][vdimp]
   pdl_launch_dependents();
@@ -227,25 +241,25 @@ __global__ void __launch_bounds__(kThreads) lm_ret_chunk_kernel(RetentionArgs a)
   const float* vb = a.qkvg + (size_t)p.row0 * a.ld + 2 * a.heads * a.dimp + h * a.vdimp;
   const int nd = min(64, a.dimp - d0), v4 = a.vdimp / 4;
   const float kscale = 1.0f / sqrtf((float)a.dim);
-  for (int i = tid; i < p.len * 16; i += kThreads) {
+  for (int i = tid; i < p.len * 16; i += kTileThreads) {
     const int j = i >> 4, c = (i & 15) * 4;
     float4 k = make_float4(0, 0, 0, 0);
     if (c < nd) k = rotated_any(kb + (size_t)j * a.ld, d0 + c, a, p.pos + j);
     const float f = pw[p.len - 1 - j] * kscale;
     *reinterpret_cast<float4*>(sK + j * 64 + c) = make_float4(k.x * f, k.y * f, k.z * f, k.w * f);
   }
-  for (int i = tid; i < p.len * v4; i += kThreads) {
+  for (int i = tid; i < p.len * v4; i += kTileThreads) {
     const int j = i / v4, c = (i - j * v4) * 4;
     *reinterpret_cast<float4*>(sV + j * a.vdimp + c) = *reinterpret_cast<const float4*>(vb + (size_t)j * a.ld + c);
   }
   __syncthreads();
   Tile<NC> acc;
   acc.clear();
-  acc.fma(sK, 64, sV, a.vdimp, p.len, ty, tx, a.vdimp);
+  acc.template fma<false>(sK, 64, sV, a.vdimp, p.len, ty, tx, a.vdimp);
   float* dst = a.chunk_state + ((size_t)chunk * a.heads + h) * a.dimp * a.vdimp;
 #pragma unroll
-  for (int r = 0; r < 4; ++r) {
-    const int d = d0 + ty * 4 + r;
+  for (int r = 0; r < kRows; ++r) {
+    const int d = d0 + ty * kRows + r;
     if (d >= a.dimp) break;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
@@ -285,18 +299,20 @@ __global__ void __launch_bounds__(kThreads) lm_ret_scan_kernel(RetentionArgs a) 
 }
 
 size_t output_smem(const RetentionArgs& a) {
-  const size_t shared_part = std::max((size_t)a.dimp * kPad, (size_t)kChunk * kPad + (size_t)2 * kStateRows * a.vdimp);
-  return ((size_t)a.dimp * kPad + shared_part + (size_t)kChunk * a.vdimp) * 4;
+  const size_t rows = (size_t)kChunk * (a.dimp + 4);
+  const size_t shared_part = std::max(rows, (size_t)kChunk * kPad + (size_t)2 * kStateRows * a.vdimp);
+  return (rows + shared_part + (size_t)kChunk * a.vdimp) * 4;
 }
 
 // grid (chunks, heads)
 template <class T, int NC>
-__global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kernel(RetentionArgs a) {
+__global__ void __launch_bounds__(kTileThreads, NC == 4 ? 1 : 2) lm_ret_output_kernel(RetentionArgs a) {
   extern __shared__ __align__(16) float out_smem[];
-  float* sQ = out_smem;                        // [dimp][kPad]: q transposed
-  float* sV = sQ + (size_t)a.dimp * kPad;      // [kChunk][vdimp]
-  float* sK = sV + (size_t)kChunk * a.vdimp;   // [dimp][kPad]: k transposed; afterwards
-  float* sA = sK;                              //   [kChunk][kPad]: decayed scores, transposed
+  const int ldq = a.dimp + 4;
+  float* sQ = out_smem;                        // [kChunk][ldq]
+  float* sV = sQ + (size_t)kChunk * ldq;       // [kChunk][vdimp]
+  float* sK = sV + (size_t)kChunk * a.vdimp;   // [kChunk][ldq]; afterwards
+  float* sA = sK;                              //   [kChunk][kPad]: decayed scores
   float* sS = sA + (size_t)kChunk * kPad;      //   [2][kStateRows][vdimp]: rows of the state
   pdl_launch_dependents();
   pdl_wait_prior();
@@ -309,45 +325,59 @@ __global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kerne
   const float* gb = vb + a.heads * a.vdimp;
   const int d4 = a.dimp / 4, v4 = a.vdimp / 4;
   const float kscale = 1.0f / sqrtf((float)a.dim);
-  for (int i = tid; i < p.len * v4; i += kThreads) {
+  for (int i = tid; i < kChunk * v4; i += kTileThreads) {
     const int j = i / v4, c = (i - j * v4) * 4;
-    cp_async16(sV + j * a.vdimp + c, vb + (size_t)j * a.ld + c);
+    if (j < p.len) cp_async16(sV + j * a.vdimp + c, vb + (size_t)j * a.ld + c);
+    else *reinterpret_cast<float4*>(sV + j * a.vdimp + c) = make_float4(0, 0, 0, 0);
   }
   asm volatile("cp.async.commit_group;" ::: "memory");
-  for (int i = tid; i < kChunk * d4; i += kThreads) {  // lanes over tokens: the transposed stores hit 32 banks
-    const int j = i & (kChunk - 1), d = (i / kChunk) * 4;
+#pragma unroll 4
+  for (int i = tid; i < kChunk * d4; i += kTileThreads) {
+    const int j = i / d4, d = (i - j * d4) * 4;
     float4 q = make_float4(0, 0, 0, 0), k = q;
     if (j < p.len) {
       q = rotated_any(qb + (size_t)j * a.ld, d, a, p.pos + j);
       k = rotated_any(kb + (size_t)j * a.ld, d, a, p.pos + j);
     }
-    sQ[d * kPad + j] = q.x, sQ[(d + 1) * kPad + j] = q.y, sQ[(d + 2) * kPad + j] = q.z, sQ[(d + 3) * kPad + j] = q.w;
-    sK[d * kPad + j] = k.x * kscale, sK[(d + 1) * kPad + j] = k.y * kscale, sK[(d + 2) * kPad + j] = k.z * kscale, sK[(d + 3) * kPad + j] = k.w * kscale;
+    *reinterpret_cast<float4*>(sQ + j * ldq + d) = q;
+    *reinterpret_cast<float4*>(sK + j * ldq + d) = make_float4(k.x * kscale, k.y * kscale, k.z * kscale, k.w * kscale);
   }
   __syncthreads();
   const float* S = a.chunk_state + ((size_t)chunk * a.heads + h) * a.dimp * a.vdimp;
   auto fetch = [&](int d0) {  // kStateRows rows of the state; dimp is a multiple of them
     float* dst = sS + (size_t)((d0 / kStateRows) & 1) * kStateRows * a.vdimp;
-    for (int i = tid; i < kStateRows * v4; i += kThreads) cp_async16(dst + 4 * i, S + (size_t)d0 * a.vdimp + 4 * i);
+    for (int i = tid; i < kStateRows * v4; i += kTileThreads) cp_async16(dst + 4 * i, S + (size_t)d0 * a.vdimp + 4 * i);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  {
-    Tile<1> s;
-    s.clear();
-    s.fma(sQ, kPad, sK, kPad, a.dimp, ty, tx, 64);
+  {  // scores of rows kRows ty .. and keys tx, tx + 16, ..; even and odd coordinates are summed side by side
+    uint64_t s[kRows][4];
+#pragma unroll
+    for (int r = 0; r < kRows; ++r) s[r][0] = s[r][1] = s[r][2] = s[r][3] = 0;
+#pragma unroll 2
+    for (int d = 0; d < a.dimp; d += 4) {
+      ulonglong2 kv[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) kv[c] = *reinterpret_cast<const ulonglong2*>(sK + (tx + 16 * c) * ldq + d);
+#pragma unroll
+      for (int r = 0; r < kRows; ++r) {
+        const ulonglong2 qv = *reinterpret_cast<const ulonglong2*>(sQ + (ty * kRows + r) * ldq + d);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          fma2(s[r][c], qv.x, kv[c].x);
+          fma2(s[r][c], qv.y, kv[c].y);
+        }
+      }
+    }
     __syncthreads();  // k is no longer needed
     fetch(0);
 #pragma unroll
-    for (int r = 0; r < 4; ++r) {
-      const float4 v = s.get(r, 0);
-      const float sv[4] = {v.x, v.y, v.z, v.w};
-      const int i = ty * 4 + r;
+    for (int r = 0; r < kRows; ++r)
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        const int j = tx * 4 + c;
-        sA[j * kPad + i] = j <= i ? sv[c] * pw[i - j] : 0.0f;
+        const int i = ty * kRows + r, j = tx + 16 * c;
+        const float2 h = halves(s[r][c]);
+        sA[i * kPad + j] = j <= i ? (h.x + h.y) * pw[i - j] : 0.0f;
       }
-    }
   }
   Tile<NC> acc;
   acc.clear();
@@ -359,15 +389,15 @@ __global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kerne
       asm volatile("cp.async.wait_group 0;" ::: "memory");
     }
     __syncthreads();
-    acc.fma(sQ + (size_t)d0 * kPad, kPad, sS + (size_t)((d0 / kStateRows) & 1) * kStateRows * a.vdimp, a.vdimp, kStateRows, ty, tx, a.vdimp);
+    acc.template fma<true>(sQ + d0, ldq, sS + (size_t)((d0 / kStateRows) & 1) * kStateRows * a.vdimp, a.vdimp, kStateRows, ty, tx, a.vdimp);
     __syncthreads();
   }
 #pragma unroll
-  for (int r = 0; r < 4; ++r) acc.scale_row(r, pw[ty * 4 + r + 1]);
-  acc.fma(sA, kPad, sV, a.vdimp, min(p.len, ty / 2 * 8 + 8), ty, tx, a.vdimp);
+  for (int r = 0; r < kRows; ++r) acc.scale_row(r, pw[ty * kRows + r + 1]);
+  acc.template fma<true>(sA, kPad, sV, a.vdimp, (ty / 2 + 1) * 2 * kRows, ty, tx, a.vdimp);
   T* out = static_cast<T*>(a.out);
 #pragma unroll
-  for (int r = 0; r < 4; ++r) {
+  for (int r = 0; r < kRows; ++r) {
     float ss = 0.0f;
 #pragma unroll
     for (int i = 0; i < NC; ++i) {
@@ -377,7 +407,7 @@ __global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kerne
     }
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    const int j = ty * 4 + r;
+    const int j = ty * kRows + r;
     if (j >= p.len) continue;
     const float inv = 1.0f / sqrtf(ss / (float)a.vdim + a.eps);
 #pragma unroll
@@ -394,12 +424,12 @@ __global__ void __launch_bounds__(kThreads, NC == 4 ? 1 : 2) lm_ret_output_kerne
 
 template <class T, int NC>
 cudaError_t prefill_nc(cudaStream_t s, const RetentionArgs& a) {
-  cudaError_t r = launch_pdl(lm_ret_chunk_kernel<NC>, dim3(a.n_chunks, a.heads, (a.dimp + 63) / 64), dim3(kThreads), (size_t)kChunk * (64 + a.vdimp) * 4, s, a);
+  cudaError_t r = launch_pdl(lm_ret_chunk_kernel<NC>, dim3(a.n_chunks, a.heads, (a.dimp + 63) / 64), dim3(kTileThreads), (size_t)kChunk * (64 + a.vdimp) * 4, s, a);
   if (r == cudaSuccess) {
     const int n4 = a.dimp * a.vdimp / 4;
     r = launch_pdl(lm_ret_scan_kernel, dim3((n4 + kThreads - 1) / kThreads, a.heads, a.n_entries), dim3(kThreads), 0, s, a);
   }
-  if (r == cudaSuccess) r = launch_pdl(lm_ret_output_kernel<T, NC>, dim3(a.n_chunks, a.heads), dim3(kThreads), output_smem(a), s, a);
+  if (r == cudaSuccess) r = launch_pdl(lm_ret_output_kernel<T, NC>, dim3(a.n_chunks, a.heads), dim3(kTileThreads), output_smem(a), s, a);
   return r;
 }
 template <class T>
