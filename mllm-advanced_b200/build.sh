@@ -10,7 +10,6 @@ NVCC="${NVCC:-/usr/local/cuda/bin/nvcc}"
 WHAT="${1:-all}"
 OUT="$HERE/lib"
 OBJ="$HERE/build"
-mkdir -p "$OUT" "$OBJ"
 CORE=(host_pack.cpp c_api.cu device_status.cu repack.cu act_quant.cu gemv.cu gemv_stream.cu gemm_stream.cu gemm_simt.cu gemm_tc.cu
       gemm_tcf16.cu decoder_kernels.cu decoder_attn.cu decoder_sample.cu decoder.cu decoder_batch.cu decoder_persistent.cu conv3d.cu
       host_pack_a16.cpp w4a16.cu c_api_a16.cu tp.cu)
@@ -26,8 +25,7 @@ compile() {
   obj="$OBJ/$(echo "$src" | tr '/.' '__').o"
   stamp="$(echo "$HEADERS ${FLAGS[*]} $(sha256sum <"$HERE/csrc/$src")" | sha256sum)"
   [ -f "$obj" ] && [ "$(cat "$obj.stamp" 2>/dev/null)" = "$stamp" ] && return 0
-  "$NVCC" "${FLAGS[@]}" -c "$HERE/csrc/$src" -o "$obj.$$.o"
-  mv "$obj.$$.o" "$obj"
+  "$NVCC" "${FLAGS[@]}" -c "$HERE/csrc/$src" -o "$obj.$$.o" && mv "$obj.$$.o" "$obj" || return 1
   echo "$stamp" >"$obj.stamp"
 }
 link() {
@@ -40,20 +38,27 @@ link() {
   echo "built $OUT/$lib"
 }
 
-case "$WHAT" in
-  all) SRC=("${CORE[@]}" "${LM[@]}") ;;
-  core) SRC=("${CORE[@]}") ;;
-  lm) SRC=("${LM[@]}") ;;
-  *) echo "usage: build.sh [all|core|lm]" >&2; exit 2 ;;
-esac
-# One build at a time; nothing to do when the libraries are those of these sources.
-exec 9>"$OBJ/.lock"
+stamp_of() { (cd "$HERE/csrc" && echo "$HEADERS ${FLAGS[*]} $(sha256sum "$@")" | sha256sum); }
+current() {  # library, its sources: built from these?
+  local lib="$1"
+  shift
+  [ -f "$OUT/$lib" ] && [ "$(cat "$OUT/.$lib.stamp" 2>/dev/null)" = "$(stamp_of "$@")" ]
+}
+todo() {
+  SRC=()
+  NEED_CORE=0
+  NEED_LM=0
+  case "$WHAT" in all | core) current libmllm_b200.so "${CORE[@]}" || { NEED_CORE=1; SRC+=("${CORE[@]}"); } ;; esac
+  case "$WHAT" in all | lm) current libmllm_b200_lm.so "${LM[@]}" || { NEED_LM=1; SRC+=("${LM[@]}"); } ;; esac
+  [ ${#SRC[@]} -gt 0 ]
+}
+
+case "$WHAT" in all | core | lm) ;; *) echo "usage: build.sh [all|core|lm]" >&2; exit 2 ;; esac
+todo || exit 0
+mkdir -p "$OUT" "$OBJ"
+exec 9>"$OBJ/.lock"  # one build at a time
 flock 9
-STAMP="$(cd "$HERE/csrc" && echo "$HEADERS ${FLAGS[*]} $(sha256sum "${SRC[@]}")" | sha256sum)"
-if [ "$(cat "$OUT/.$WHAT.stamp" 2>/dev/null)" = "$STAMP" ] && { [ "$WHAT" = lm ] || [ -f "$OUT/libmllm_b200.so" ]; } &&
-   { [ "$WHAT" = core ] || [ -f "$OUT/libmllm_b200_lm.so" ]; }; then
-  exit 0
-fi
+todo || exit 0
 JOBS="$(nproc)"
 rm -f "$OBJ/.failed"
 declare -A started=()
@@ -65,6 +70,11 @@ for s in "${SRC[@]}"; do
 done
 wait
 [ ! -e "$OBJ/.failed" ] || { echo "build.sh: a source did not compile" >&2; exit 1; }
-[ "$WHAT" = lm ] || link libmllm_b200.so "${CORE[@]}"
-[ "$WHAT" = core ] || link libmllm_b200_lm.so "${LM[@]}"
-echo "$STAMP" >"$OUT/.$WHAT.stamp"
+finish() {
+  link "$@"
+  local lib="$1"
+  shift
+  stamp_of "$@" >"$OUT/.$lib.stamp"
+}
+[ "$NEED_CORE" = 0 ] || finish libmllm_b200.so "${CORE[@]}"
+[ "$NEED_LM" = 0 ] || finish libmllm_b200_lm.so "${LM[@]}"
