@@ -14,12 +14,12 @@ CORE=(host_pack.cpp c_api.cu device_status.cu repack.cu act_quant.cu gemv.cu gem
       gemm_tcf16.cu decoder_kernels.cu decoder_attn.cu decoder_sample.cu decoder.cu decoder_batch.cu decoder_persistent.cu conv3d.cu
       host_pack_a16.cpp w4a16.cu c_api_a16.cu tp.cu)
 [ -f "$HERE/csrc/no_alloc.cu" ] && CORE+=(no_alloc.cu)
-LM=(lm/lm_engine.cu lm/lm_linear.cu lm/lm_norm.cu lm/lm_attn.cu lm/lm_retention.cu device_status.cu decoder_sample.cu)
+LM=(lm/lm_engine.cu lm/lm_linear.cu lm/lm_norm.cu lm/lm_attn.cu lm/lm_latent.cu lm/lm_moe.cu lm/lm_retention.cu device_status.cu decoder_sample.cu)
 FLAGS=(-std=c++17 -O3 -gencode arch=compute_100a,code=sm_100a -lineinfo -rdc=true -Xcompiler -fPIC,-fvisibility=hidden,-O3)
 [ -n "${PTXAS_V:-}" ] && FLAGS+=(-Xptxas -v)
 
 # what an object depends on: every header, its own source, the flags
-HEADERS="$(cat "$HERE"/csrc/*.h "$HERE"/csrc/*.cuh "$HERE"/csrc/*.inc "$HERE"/csrc/lm/*.h "$HERE"/../include/*.h | sha256sum)"
+HEADERS="$(cat "$HERE"/csrc/*.h "$HERE"/csrc/*.cuh "$HERE"/csrc/*.inc "$HERE"/csrc/lm/*.h "$HERE"/csrc/lm/*.cuh "$HERE"/../include/*.h | sha256sum)"
 compile() {
   local src="$1" obj stamp
   obj="$OBJ/$(echo "$src" | tr '/.' '__').o"

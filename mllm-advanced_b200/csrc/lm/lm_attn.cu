@@ -1,4 +1,5 @@
-// Softmax attention of the language-model engine over slot caches [slot][kv_heads][max_ctx][dim], with grouped query
+// Softmax attention of the language-model engine over keys and values in rows per head (slot caches
+// [slot][kv_heads][max_ctx][dim], or keys and values made from latents for one step), with grouped query
 // heads, a learned distance bias (a table per layer and head, indexed by min(distance, bias_max)) and an optional sink:
 // a key of score 0 without a value, i.e. one more term exp(0) in the denominator.  Keys and values of the step are in
 // the caches already.  Scores, weights and sums are fp32; the bf16 kernels multiply bf16 queries and keys exactly into
@@ -23,18 +24,20 @@ constexpr float kNegInf = -3.402823466e+38f;
 // ------------------------------------------------------------------------------------------ fp32, any row
 constexpr int kF32Threads = 128;
 
+// NV: value columns per thread
+template <int NV>
 __global__ void __launch_bounds__(kF32Threads) lm_attn_f32_kernel(AttnShape a, const float* __restrict__ q, int ldq,
                                                                   const int2* __restrict__ row_sp, const float* __restrict__ kc,
                                                                   const float* __restrict__ vc, const float* __restrict__ bias,
                                                                   float* __restrict__ out, int ldo) {
-  __shared__ __align__(16) float sq[256], sp[kF32Threads], red[kF32Threads / 32];
+  __shared__ __align__(16) float sq[1024], sp[kF32Threads], red[kF32Threads / 32];
   pdl_launch_dependents();
   pdl_wait_prior();
   const int row = blockIdx.x, h = blockIdx.y, g = h / (a.heads / a.kv_heads), tid = threadIdx.x;
   const int2 s = row_sp[row];
-  const size_t base = ((size_t)s.x * a.kv_heads + g) * a.max_ctx;
+  const size_t base = s.x * a.slot_rows + g * a.head_rows;
   for (int d = tid; d < a.dimp; d += kF32Threads) sq[d] = q[(size_t)row * ldq + h * a.dimp + d];
-  float m = a.sink ? 0.0f : kNegInf, l = a.sink ? 1.0f : 0.0f, acc[2] = {0.0f, 0.0f};
+  float m = a.sink ? 0.0f : kNegInf, l = a.sink ? 1.0f : 0.0f, acc[NV] = {};
   auto block_reduce = [&](float v, bool is_max) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
@@ -67,7 +70,7 @@ __global__ void __launch_bounds__(kF32Threads) lm_attn_f32_kernel(AttnShape a, c
     m = m_new;
     const int nk = min(kF32Threads, s.y + 1 - j0);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
+    for (int i = 0; i < NV; ++i) {
       const int d = tid + i * kF32Threads;
       if (d < a.vdimp) {
         float o = acc[i] * alpha;
@@ -78,7 +81,7 @@ __global__ void __launch_bounds__(kF32Threads) lm_attn_f32_kernel(AttnShape a, c
     __syncthreads();
   }
 #pragma unroll
-  for (int i = 0; i < 2; ++i) {
+  for (int i = 0; i < NV; ++i) {
     const int d = tid + i * kF32Threads;
     if (d < a.vdimp) out[(size_t)row * ldo + h * a.vdimp + d] = acc[i] / l;
   }
@@ -152,8 +155,8 @@ __global__ void __launch_bounds__(kPfThreads) lm_attn_prefill_kernel(AttnShape a
   const int4 tile = tiles[blockIdx.x];
   const int kvh = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = warp >> 2, wrow = (warp & 3) * 16;
   const int row0 = tile.x, ntok = tile.y, pos0 = tile.w, last = pos0 + ntok - 1;
-  const __nv_bfloat16* kb = kc + ((size_t)tile.z * a.kv_heads + kvh) * a.max_ctx * D;
-  const __nv_bfloat16* vb = vc + ((size_t)tile.z * a.kv_heads + kvh) * a.max_ctx * a.vdimp;
+  const __nv_bfloat16* kb = kc + (tile.z * a.slot_rows + kvh * a.head_rows) * D;
+  const __nv_bfloat16* vb = vc + (tile.z * a.slot_rows + kvh * a.head_rows) * a.vdimp;
   const int dv8 = D / 8, vv8 = a.vdimp / 8;
   // copies: eight threads per row of 16-byte pieces
   const int cr = tid >> 3, cc = tid & 7;
@@ -361,7 +364,7 @@ __global__ void __launch_bounds__(kDecThreads) lm_attn_decode_kernel(AttnShape a
   const int j0 = split * kKeys, nk = min(kKeys, sp.y + 1 - j0);
   if (nk <= 0) return;
   const int nh = min(kDecRows, group - hb0), h0 = kvh * group + hb0, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const size_t base = ((size_t)sp.x * a.kv_heads + kvh) * a.max_ctx + j0;
+  const size_t base = sp.x * a.slot_rows + kvh * a.head_rows + j0;
   const int dv8 = D / 8, vv8 = a.vdimp / 8;
   const int cr = tid >> 3, cc = tid & 7;  // copies: eight threads per row of 16-byte pieces
   for (int c = cc; c < dv8; c += 8)
@@ -566,9 +569,13 @@ cudaError_t attention_configure() {
 cudaError_t launch_attention(cudaStream_t s, bool f32, const AttnShape& a, const void* q, int ldq, const int2* row_sp, int rows,
                              const void* kc, const void* vc, const float* bias, void* out, int ldo, const int4* tiles, int n_tiles,
                              const int* single_rows, int n_single, int chunk, int splits, float* part_o, float2* part_ml) {
-  if (f32)
-    return launch_pdl(lm_attn_f32_kernel, dim3(rows, a.heads), dim3(kF32Threads), 0, s, a, static_cast<const float*>(q), ldq, row_sp,
-                      static_cast<const float*>(kc), static_cast<const float*>(vc), bias, static_cast<float*>(out), ldo);
+  if (f32) {
+    auto go = [&](auto f) {
+      return launch_pdl(f, dim3(rows, a.heads), dim3(kF32Threads), 0, s, a, static_cast<const float*>(q), ldq, row_sp,
+                        static_cast<const float*>(kc), static_cast<const float*>(vc), bias, static_cast<float*>(out), ldo);
+    };
+    return a.vdimp <= 2 * kF32Threads ? go(lm_attn_f32_kernel<2>) : go(lm_attn_f32_kernel<8>);
+  }
   const auto* qb = static_cast<const __nv_bfloat16*>(q);
   const auto *kb = static_cast<const __nv_bfloat16*>(kc), *vb = static_cast<const __nv_bfloat16*>(vc);
   auto* ob = static_cast<__nv_bfloat16*>(out);

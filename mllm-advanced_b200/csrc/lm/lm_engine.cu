@@ -4,7 +4,9 @@
 // A step is a ragged batch: rows (tokens) of several sequences, one after the other.  Linears and norms see rows;
 // attention, retention and the convolution see sequences through row and entry tables in device memory.  A layer is
 //   norm + conv | in-projection | mixer | out-projection | norm | gate-up | down
-// where every norm also folds in the residual: x' = x + post_norm(sublayer), h = pre_norm(x').
+// where every norm also folds in the residual: x' = x + post_norm(sublayer), h = pre_norm(x'); or, with the norms behind
+// the residual sum,
+//   in-projection | mixer | out-projection | norm (+ choice of experts) | gate-up | down | norm.
 #include <algorithm>
 #include <cmath>
 #include <cstdarg>
@@ -26,6 +28,13 @@ constexpr int kArgmaxBlocks = 32;
 struct GraphKey {
   int count, chunk, splits;
   bool operator<(const GraphKey& o) const { return std::tie(count, chunk, splits) < std::tie(o.count, o.chunk, o.splits); }
+};
+// Sequences whose keys and values are made from latents together: their row tiles of the cache (per layer the same) and
+// the attention tiles over the result.
+struct ExpandPass {
+  const int4* rows = nullptr;
+  const int4* tiles = nullptr;
+  int n_rows = 0, n_tiles = 0, total = 0;
 };
 // Positions per CTA of the decode attention: small pieces while they are needed to fill the GPU.
 int decode_chunk(int sequences, int longest) {
@@ -49,11 +58,15 @@ struct StepCtx {
   std::map<int, std::pair<const int4*, int>> tiles;
   const int2 *chunks = nullptr, *entry_chunks = nullptr;
   int n_chunks = 0;
+  // latent attention: rows that attend through the latent (nullptr: all), a bound of their contexts, and the others
+  const int* latent_rows = nullptr;
+  int n_latent = 0, latent_ctx = 1;
+  std::vector<ExpandPass> expand;
 };
 
 struct Engine {
   mllmb200_lm_config c{};
-  bool f32 = false;
+  bool f32 = false, post = false, latent = false;
   int elt = 2, widthp = 0, plane_rows = 0, logit_rows = 0, max_splits_ctx = 1;
   std::vector<LayerState> layers;
   __nv_bfloat16* embed = nullptr;
@@ -63,6 +76,18 @@ struct Engine {
   // activations
   float *xa = nullptr, *xb = nullptr, *delta = nullptr, *proj = nullptr, *logits = nullptr, *chunk_state = nullptr, *part_o = nullptr;
   float2 *part_ml = nullptr, *best = nullptr;
+  // latent attention: rows before their norm, queries against the latent and outputs in it, keys and values of a step
+  float *fresh = nullptr, *lat = nullptr, *lat_part = nullptr;
+  float2* lat_ml = nullptr;
+  void *qa = nullptr, *ex_k = nullptr, *ex_v = nullptr;
+  int latent_cap = 0, expand_cap = 0;
+  // experts
+  float *route_logits = nullptr, *route_weight = nullptr;
+  int *route_sel = nullptr, *route_rank = nullptr, *route_count = nullptr, *pair_row = nullptr, *n_moe_tiles = nullptr;
+  int4* moe_tiles = nullptr;
+  void* permuted = nullptr;
+  ActMap m_permuted;
+  int n_route_count = 0, route_planes = 1;
   void *h = nullptr, *mix = nullptr, *act = nullptr, *hf = nullptr;
   ActMap m_h, m_hf;
   // bookkeeping: the host's view of every slot, and the device's for decode graphs
@@ -125,15 +150,18 @@ int dalloc_bytes(Engine* e, void** p, size_t bytes, bool state = false) {
   *p = q;
   return MLLMB200_OK;
 }
-int make_linear(Engine* e, Linear* l, int n, int k) {
+int make_linear(Engine* e, Linear* l, int n, int k, int groups = 1) {
   l->n = n;
   l->k = pad_to(k, 64);
-  LM_OK(dalloc(e, &l->w, (size_t)n * l->k));
+  l->groups = groups;
+  LM_OK(dalloc(e, &l->w, (size_t)groups * n * l->k));
   if (make_linear_maps(l) != MLLMB200_OK) return fail(e, MLLMB200_CUDA_ERROR, "tensor map of a [%d, %d] weight", n, l->k);
   return MLLMB200_OK;
 }
 
 bool is_attn(const LayerState& L) { return L.d.mixer == MLLMB200_LM_ATTENTION; }
+bool is_latent(const LayerState& L) { return L.d.mixer == MLLMB200_LM_LATENT; }
+bool owns_latent(const LayerState& L) { return is_latent(L) && L.d.kv_from < 0; }
 int qk_cols(const LayerState& L) { return L.d.heads * L.dimp; }
 int mix_cols(const LayerState& L) { return L.d.heads * L.vdimp; }
 
@@ -148,11 +176,31 @@ int bucket_of(int n, int rows, int max_distance) {
   return std::min(rows - 1, half + m);
 }
 
+int check_latent(Engine* e, int i, const mllmb200_lm_layer& d) {
+  if (d.kv_rank < 1) return fail(e, MLLMB200_INVALID_ARG, "layer %d: size of the latent", i);
+  if (d.kv_rank > kMaxRank) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: latents beyond %d", i, kMaxRank);
+  if (d.kv_heads != d.heads) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: latent attention has as many key as query heads", i);
+  if (d.rot_dims || d.bias_rows || d.sink || d.weights_of >= 0)
+    return fail(e, MLLMB200_UNSUPPORTED, "layer %d: rotation, distance bias, sink or shared weights in latent attention", i);
+  if (e->c.max_rows > 65535) return fail(e, MLLMB200_UNSUPPORTED, "more than 65535 rows in a step of latent attention");
+  if (d.kv_from < 0) return MLLMB200_OK;
+  if (d.kv_from >= i || !owns_latent(e->layers[d.kv_from]) || e->layers[d.kv_from].d.kv_rank != d.kv_rank)
+    return fail(e, MLLMB200_INVALID_ARG, "layer %d: layer %d has no cache of its own with latents of %d", i, d.kv_from, d.kv_rank);
+  return MLLMB200_OK;
+}
+
 int check_layer(Engine* e, int i, const mllmb200_lm_layer& d) {
-  if (d.mixer != MLLMB200_LM_ATTENTION && d.mixer != MLLMB200_LM_RETENTION) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: mixer %d", i, d.mixer);
+  if (d.mixer != MLLMB200_LM_ATTENTION && d.mixer != MLLMB200_LM_RETENTION && d.mixer != MLLMB200_LM_LATENT)
+    return fail(e, MLLMB200_UNSUPPORTED, "layer %d: mixer %d", i, d.mixer);
   if (d.heads < 1 || d.kv_heads < 1 || d.heads % d.kv_heads || d.dim < 1 || d.vdim < 1 || d.ff < 0)
     return fail(e, MLLMB200_INVALID_ARG, "layer %d: sizes", i);
   if (d.dim > 256 || d.vdim > 256 || d.heads / d.kv_heads > 64) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: head sizes beyond 256 or more than 64 heads per key", i);
+  if (d.act < MLLMB200_LM_ACT_CLAMPED || d.act > MLLMB200_LM_ACT_SILU) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: activation %d", i, d.act);
+  if (d.experts) {
+    if (d.experts < 1 || d.top < 1 || d.top > d.experts || d.ff < 1) return fail(e, MLLMB200_INVALID_ARG, "layer %d: %d of %d experts", i, d.top, d.experts);
+    if (d.experts > kMaxExperts || d.top > kMaxTop) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: more than %d experts or %d at a time", i, kMaxExperts, kMaxTop);
+  }
+  if (d.mixer == MLLMB200_LM_LATENT) return check_latent(e, i, d);
   if (d.mixer == MLLMB200_LM_RETENTION) {
     if (d.kv_heads != d.heads) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: retention has as many key as query heads", i);
     if (d.rot_dims < 0 || d.rot_dims % 2 || d.rot_dims > d.dim || (d.rot_dims && !(d.rot_base > 0))) return fail(e, MLLMB200_INVALID_ARG, "layer %d: rotation", i);
@@ -163,10 +211,9 @@ int check_layer(Engine* e, int i, const mllmb200_lm_layer& d) {
   }
   if (d.weights_of >= 0) {
     if (d.weights_of >= i) return fail(e, MLLMB200_INVALID_ARG, "layer %d: weights of a later layer", i);
-    mllmb200_lm_layer o = e->layers[d.weights_of].d, m = d;
-    o.weights_of = m.weights_of = -1;
+    const mllmb200_lm_layer &o = e->layers[d.weights_of].d, &m = d;
     if (o.mixer != m.mixer || o.heads != m.heads || o.kv_heads != m.kv_heads || o.dim != m.dim || o.vdim != m.vdim || o.ff != m.ff ||
-        o.bias_rows != m.bias_rows || o.bias_max != m.bias_max)
+        o.bias_rows != m.bias_rows || o.bias_max != m.bias_max || o.experts != m.experts)
       return fail(e, MLLMB200_INVALID_ARG, "layer %d differs from layer %d, whose weights it uses", i, d.weights_of);
   }
   return MLLMB200_OK;
@@ -175,8 +222,11 @@ int check_layer(Engine* e, int i, const mllmb200_lm_layer& d) {
 int create(Engine* e, const mllmb200_lm_layer* descs) {
   const auto& c = e->c;
   if (c.vocab < 1 || c.width < 1 || c.layers < 1 || c.conv_taps < 0 || c.max_seqs < 1 || c.max_ctx < 1 || c.max_rows < 1 ||
-      (c.dtype != MLLMB200_LM_BF16 && c.dtype != MLLMB200_LM_F32))
+      (c.dtype != MLLMB200_LM_BF16 && c.dtype != MLLMB200_LM_F32) ||
+      (c.norm_place != MLLMB200_LM_NORM_SANDWICH && c.norm_place != MLLMB200_LM_NORM_POST))
     return fail(e, MLLMB200_INVALID_ARG, "model sizes");
+  e->post = c.norm_place == MLLMB200_LM_NORM_POST;
+  if (e->post && c.conv_taps) return fail(e, MLLMB200_UNSUPPORTED, "an input convolution with norms behind the residual sum");
   e->f32 = c.dtype == MLLMB200_LM_F32;
   e->elt = e->f32 ? 4 : 2;
   e->widthp = pad_to(c.width, 64);
@@ -186,15 +236,17 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
   LM_CUDA(linear_configure());
   LM_CUDA(attention_configure());
   LM_CUDA(retention_configure());
+  LM_CUDA(latent_configure());
   const size_t rows = c.max_rows, slots = c.max_seqs;
   e->plane_rows = std::max(c.max_rows, 1024);
   e->logit_rows = std::max(std::min(c.max_rows, 128), c.max_seqs);
   e->max_splits_ctx = (c.max_ctx + kMinDecodeChunk - 1) / kMinDecodeChunk;
   LM_OK(dalloc(e, &e->embed, (size_t)c.vocab * c.width));
   LM_OK(make_linear(e, &e->head, c.vocab, c.width));
-  LM_OK(dalloc(e, &e->final_gain, 1));
+  LM_OK(dalloc(e, &e->final_gain, e->post ? e->widthp : 1));
   std::map<std::pair<int, double>, std::pair<float*, float*>> ropes;
   size_t proj_bytes = 0, mix_elems = 0, act_elems = 0, part = 0, heads = 0, chunk_elems = 0;
+  size_t rank = 0, head_rank = 0, lat_heads = 0, ex_k = 0, ex_v = 0, experts = 0, top = 0;
   e->layers.resize(c.layers);
   for (int i = 0; i < c.layers; ++i) {
     LayerState& L = e->layers[i];
@@ -203,19 +255,32 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
     L.src = L.d.weights_of < 0 ? i : e->layers[L.d.weights_of].src;
     L.dimp = pad_to(L.d.dim, 16);
     L.vdimp = pad_to(L.d.vdim, 16);
+    L.rankp = is_latent(L) ? pad_to(L.d.kv_rank, 64) : 0;
     const int G = L.d.kv_heads;
     if (L.src == i) {
-      const int n_in = is_attn(L) ? qk_cols(L) + G * (L.dimp + L.vdimp) : 2 * (qk_cols(L) + mix_cols(L));
+      const int n_in = is_attn(L)     ? qk_cols(L) + G * (L.dimp + L.vdimp)
+                       : is_latent(L) ? qk_cols(L) + (owns_latent(L) ? L.rankp : 0)
+                                      : 2 * (qk_cols(L) + mix_cols(L));
       LM_OK(make_linear(e, &L.w.in, n_in, c.width));
       LM_OK(make_linear(e, &L.w.out, c.width, mix_cols(L)));
       if (L.d.ff) {
-        LM_OK(make_linear(e, &L.w.gate_up, 2 * L.d.ff, c.width));
-        LM_OK(make_linear(e, &L.w.down, c.width, L.d.ff));
+        LM_OK(make_linear(e, &L.w.gate_up, 2 * L.d.ff, c.width, std::max(1, L.d.experts)));
+        LM_OK(make_linear(e, &L.w.down, c.width, L.d.ff, std::max(1, L.d.experts)));
       }
-      LM_OK(dalloc(e, &L.w.norms, 4));
+      if (L.d.experts) {
+        LM_OK(make_linear(e, &L.w.router, L.d.experts, c.width));
+        LM_OK(dalloc(e, &L.w.router_b, L.d.experts));
+        L.w.expert_loaded.assign(L.d.experts, 0);
+      }
+      if (is_latent(L)) {
+        LM_OK(make_linear(e, &L.w.uk_uv, qk_cols(L) + mix_cols(L), L.d.kv_rank));
+        LM_OK(dalloc(e, &L.w.uk_t, (size_t)L.d.heads * L.rankp * L.dimp));
+        if (owns_latent(L)) LM_OK(dalloc(e, &L.w.kv_gain, L.rankp));
+      }
+      LM_OK(dalloc(e, &L.w.norms, e->post ? 2 * (size_t)e->widthp : 4));
       if (c.conv_taps) LM_OK(dalloc(e, &L.w.conv, (size_t)c.conv_taps * e->widthp));
       if (is_attn(L) && L.d.bias_rows) LM_OK(dalloc(e, &L.w.bias, (size_t)L.d.heads * (L.d.bias_max + 1)));
-      if (!is_attn(L)) LM_OK(dalloc(e, &L.w.decay, (size_t)L.d.heads * (kChunk + 1)));
+      if (L.d.mixer == MLLMB200_LM_RETENTION) LM_OK(dalloc(e, &L.w.decay, (size_t)L.d.heads * (kChunk + 1)));
     }
     if (is_attn(L)) {
       LM_OK(dalloc_bytes(e, &L.kc, slots * G * c.max_ctx * L.dimp * e->elt, true));
@@ -223,6 +288,21 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
       proj_bytes = std::max(proj_bytes, rows * qk_cols(L) * e->elt);
       part = std::max(part, (size_t)mix_cols(L));
       heads = std::max(heads, (size_t)L.d.heads);
+    } else if (is_latent(L)) {
+      e->latent = true;
+      if (owns_latent(L)) {
+        LM_OK(dalloc_bytes(e, &L.kc, slots * c.max_ctx * L.rankp * e->elt, true));
+        if (make_act_map(&L.a_kc, L.kc, (int)(slots * c.max_ctx), L.rankp) != MLLMB200_OK) return fail(e, MLLMB200_CUDA_ERROR, "tensor map of a latent cache");
+      } else {
+        L.kc = e->layers[L.d.kv_from].kc;
+        L.a_kc = e->layers[L.d.kv_from].a_kc;
+      }
+      proj_bytes = std::max(proj_bytes, rows * qk_cols(L) * e->elt);
+      rank = std::max(rank, (size_t)L.rankp);
+      head_rank = std::max(head_rank, (size_t)L.d.heads * L.rankp);
+      lat_heads = std::max(lat_heads, (size_t)L.d.heads);
+      ex_k = std::max(ex_k, (size_t)qk_cols(L));
+      ex_v = std::max(ex_v, (size_t)mix_cols(L));
     } else {
       LM_OK(dalloc(e, &L.state, slots * L.d.heads * L.dimp * L.vdimp, true));
       proj_bytes = std::max(proj_bytes, rows * 2 * (size_t)(qk_cols(L) + mix_cols(L)) * 4);
@@ -241,7 +321,39 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
     }
     if (c.conv_taps > 1) LM_OK(dalloc(e, &L.tail, slots * 2 * (c.conv_taps - 1) * e->widthp, true));
     mix_elems = std::max(mix_elems, rows * (size_t)pad_to(mix_cols(L), 64));
-    if (L.d.ff) act_elems = std::max(act_elems, rows * (size_t)pad_to(L.d.ff, 64));
+    if (L.d.ff) act_elems = std::max(act_elems, rows * (L.d.experts ? L.d.top : 1) * (size_t)pad_to(L.d.ff, 64));
+    experts = std::max(experts, (size_t)L.d.experts);
+    top = std::max(top, (size_t)L.d.top * (L.d.experts ? 1 : 0));
+  }
+  e->plane_rows = std::max(e->plane_rows, (int)(rows * top));
+  if (e->latent) {
+    e->latent_cap = e->f32 ? c.max_rows : std::min(c.max_rows, c.max_seqs * kAbsorbMax);
+    LM_OK(dalloc(e, &e->fresh, rows * rank));
+    LM_OK(dalloc_bytes(e, &e->qa, e->latent_cap * head_rank * e->elt));
+    if (e->f32) {
+      LM_OK(dalloc(e, &e->lat, rows * head_rank));
+    } else {
+      LM_OK(dalloc(e, &e->lat_part, latent_parts(e->latent_cap) * head_rank));
+      LM_OK(dalloc(e, &e->lat_ml, latent_parts(e->latent_cap) * lat_heads));
+      e->expand_cap = c.max_ctx + (c.max_seqs > 1 ? c.max_rows : 0);
+      LM_OK(dalloc_bytes(e, &e->ex_k, e->expand_cap * ex_k * e->elt));
+      LM_OK(dalloc_bytes(e, &e->ex_v, e->expand_cap * ex_v * e->elt));
+    }
+  }
+  if (experts) {
+    const size_t pairs = rows * top;
+    e->n_route_count = (int)(c.layers * experts);
+    e->route_planes = kMaxSplits;
+    LM_OK(dalloc(e, &e->route_logits, rows * pad_to((int)experts, 4) * e->route_planes));
+    LM_OK(dalloc(e, &e->route_weight, pairs));
+    LM_OK(dalloc(e, &e->route_sel, pairs));
+    LM_OK(dalloc(e, &e->route_rank, pairs));
+    LM_OK(dalloc(e, &e->pair_row, pairs));
+    LM_OK(dalloc(e, &e->route_count, e->n_route_count));
+    LM_OK(dalloc(e, &e->n_moe_tiles, 1));
+    LM_OK(dalloc(e, &e->moe_tiles, experts + pairs / group_tile_rows(e->f32) + 1));
+    LM_OK(dalloc_bytes(e, &e->permuted, pairs * e->widthp * e->elt));
+    if (make_act_map(&e->m_permuted, e->permuted, (int)pairs, e->widthp) != MLLMB200_OK) return fail(e, MLLMB200_CUDA_ERROR, "tensor map of the activations");
   }
   LM_OK(dalloc(e, &e->xa, rows * e->widthp));
   LM_OK(dalloc(e, &e->xb, rows * e->widthp));
@@ -262,7 +374,7 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
     return fail(e, MLLMB200_CUDA_ERROR, "tensor map of the activations");
   for (auto& L : e->layers) {
     bool ok = make_act_map(&L.a_mix, e->mix, c.max_rows, pad_to(mix_cols(L), 64)) == MLLMB200_OK;
-    if (L.d.ff) ok = ok && make_act_map(&L.a_act, e->act, c.max_rows, pad_to(L.d.ff, 64)) == MLLMB200_OK;
+    if (L.d.ff) ok = ok && make_act_map(&L.a_act, e->act, c.max_rows * (L.d.experts ? L.d.top : 1), pad_to(L.d.ff, 64)) == MLLMB200_OK;
     if (!ok) return fail(e, MLLMB200_CUDA_ERROR, "tensor map of the activations");
   }
   LM_OK(dalloc(e, &e->d_pos, slots));
@@ -317,6 +429,31 @@ int to_device(Engine* e, T* dst, const std::vector<T>& v) {
   return MLLMB200_OK;
 }
 
+// A tensor's rows to one group of a linear, row r to r row_mul + row_off.
+int pack_group(Engine* e, const Linear& l, int group, int row_mul, int row_off, const void* data, int rows, int cols) {
+  Linear g = l;
+  g.w = l.w + (size_t)group * l.n * l.k;
+  return pack(e, {&g, rows, cols, rows, rows, row_mul, row_off, cols, cols}, data);
+}
+int set_vector(Engine* e, float* dst, const void* data, int n) {
+  LM_CUDA(cudaMemcpy(dst, data, (size_t)n * 4, cudaMemcpyDefault));
+  return MLLMB200_OK;
+}
+
+int set_expert(Engine* e, int layer, int expert, int which, const void* data, int rows, int cols) {
+  if (layer < 0 || layer >= e->c.layers || e->layers[layer].src != layer || expert < 0 || expert >= e->layers[layer].d.experts)
+    return fail(e, MLLMB200_INVALID_ARG, "expert %d of layer %d", expert, layer);
+  LayerState& L = e->layers[layer];
+  const bool down = which == MLLMB200_LM_T_DOWN;
+  const int n = down ? e->c.width : L.d.ff, k = down ? L.d.ff : e->c.width;
+  if ((!down && which != MLLMB200_LM_T_GATE && which != MLLMB200_LM_T_UP) || rows != n || cols != k)
+    return fail(e, MLLMB200_INVALID_ARG, "tensor %d of expert %d of layer %d is [%d, %d], expected [%d, %d]", which, expert, layer, rows, cols, n, k);
+  if (down) LM_OK(pack_group(e, L.w.down, expert, 1, 0, data, rows, cols));
+  else LM_OK(pack_group(e, L.w.gate_up, expert, 2, which == MLLMB200_LM_T_UP, data, rows, cols));
+  L.w.expert_loaded[expert] |= 1u << which;
+  return MLLMB200_OK;
+}
+
 int set_tensor(Engine* e, int layer, int which, const void* data, int rows, int cols) {
   const auto& c = e->c;
   auto shape = [&](int r, int k) {
@@ -331,8 +468,8 @@ int set_tensor(Engine* e, int layer, int which, const void* data, int rows, int 
       LM_OK(shape(c.vocab, c.width));
       LM_OK(pack(e, {&e->head, rows, cols, rows, rows, 1, 0, cols, cols}, data));
     } else if (which == MLLMB200_LM_T_FINAL_NORM) {
-      LM_OK(shape(1, 1));
-      LM_CUDA(cudaMemcpy(e->final_gain, data, 4, cudaMemcpyDefault));
+      LM_OK(shape(1, e->post ? c.width : 1));
+      LM_OK(set_vector(e, e->final_gain, data, cols));
     } else {
       return fail(e, MLLMB200_INVALID_ARG, "tensor %d", which);
     }
@@ -349,16 +486,58 @@ int set_tensor(Engine* e, int layer, int which, const void* data, int rows, int 
       LM_OK(shape(H * d.dim, c.width));
       LM_OK(pack(e, {&L.w.in, rows, cols, d.dim, L.dimp, 1, 0, cols, cols}, data));
       break;
+    case MLLMB200_LM_T_DKV:
+      if (!owns_latent(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d makes no latents", layer);
+      LM_OK(shape(d.kv_rank, c.width));
+      LM_OK(pack(e, {&L.w.in, rows, cols, rows, rows, 1, qk_cols(L), cols, cols}, data));
+      break;
+    case MLLMB200_LM_T_DKV_NORM:
+      if (!owns_latent(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d makes no latents", layer);
+      LM_OK(shape(1, d.kv_rank));
+      LM_OK(set_vector(e, L.w.kv_gain, data, cols));
+      break;
+    case MLLMB200_LM_T_UK: {
+      if (!is_latent(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no latent attention", layer);
+      LM_OK(shape(H * d.dim, d.kv_rank));
+      LM_OK(pack(e, {&L.w.uk_uv, rows, cols, d.dim, L.dimp, 1, 0, cols, cols}, data));
+      std::vector<uint16_t> src;
+      LM_OK(to_host(e, &src, data, (size_t)rows * cols));
+      __nv_bfloat16* staged = nullptr;
+      LM_CUDA(cudaMalloc(reinterpret_cast<void**>(&staged), src.size() * 2));
+      cudaError_t r = cudaMemcpyAsync(staged, src.data(), src.size() * 2, cudaMemcpyHostToDevice, e->stream);
+      if (r == cudaSuccess) r = launch_pack_heads_transposed(e->stream, staged, H, d.dim, d.kv_rank, L.w.uk_t, L.rankp, L.dimp);
+      if (r == cudaSuccess) r = cudaStreamSynchronize(e->stream);
+      cudaFree(staged);
+      LM_CUDA(r);
+      break;
+    }
+    case MLLMB200_LM_T_UV:
+      if (!is_latent(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no latent attention", layer);
+      LM_OK(shape(H * d.vdim, d.kv_rank));
+      LM_OK(pack(e, {&L.w.uk_uv, rows, cols, d.vdim, L.vdimp, 1, qk_cols(L), cols, cols}, data));
+      break;
+    case MLLMB200_LM_T_ROUTER:
+      if (!d.experts) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no experts", layer);
+      LM_OK(shape(d.experts, c.width));
+      LM_OK(pack(e, {&L.w.router, rows, cols, rows, rows, 1, 0, cols, cols}, data));
+      break;
+    case MLLMB200_LM_T_ROUTER_B:
+      if (!d.experts) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no experts", layer);
+      LM_OK(shape(1, d.experts));
+      LM_OK(set_vector(e, L.w.router_b, data, cols));
+      break;
     case MLLMB200_LM_T_K:
+      if (is_latent(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d makes its keys from latents", layer);
       LM_OK(shape(G * d.dim, c.width));
       LM_OK(pack(e, {&L.w.in, rows, cols, d.dim, L.dimp, 1, k_off, cols, cols}, data));
       break;
     case MLLMB200_LM_T_V:
+      if (is_latent(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d makes its values from latents", layer);
       LM_OK(shape(G * d.vdim, c.width));
       LM_OK(pack(e, {&L.w.in, rows, cols, d.vdim, L.vdimp, 1, v_off, cols, cols}, data));
       break;
     case MLLMB200_LM_T_G:
-      if (is_attn(L)) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no output gate", layer);
+      if (!L.w.decay) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no output gate", layer);
       LM_OK(shape(H * d.vdim, c.width));
       LM_OK(pack(e, {&L.w.in, rows, cols, d.vdim, L.vdimp, 1, g_off, cols, cols}, data));
       break;
@@ -368,12 +547,12 @@ int set_tensor(Engine* e, int layer, int which, const void* data, int rows, int 
       break;
     case MLLMB200_LM_T_GATE:
     case MLLMB200_LM_T_UP:
-      if (!d.ff) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no feed-forward", layer);
+      if (!d.ff || d.experts) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no dense feed-forward", layer);
       LM_OK(shape(d.ff, c.width));
       LM_OK(pack(e, {&L.w.gate_up, rows, cols, rows, rows, 2, which == MLLMB200_LM_T_UP, cols, cols}, data));
       break;
     case MLLMB200_LM_T_DOWN:
-      if (!d.ff) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no feed-forward", layer);
+      if (!d.ff || d.experts) return fail(e, MLLMB200_INVALID_ARG, "layer %d has no dense feed-forward", layer);
       LM_OK(shape(c.width, d.ff));
       LM_OK(pack(e, {&L.w.down, rows, cols, rows, rows, 1, 0, cols, cols}, data));
       break;
@@ -381,8 +560,14 @@ int set_tensor(Engine* e, int layer, int which, const void* data, int rows, int 
     case MLLMB200_LM_T_NORM1B:
     case MLLMB200_LM_T_NORM2:
     case MLLMB200_LM_T_NORM2B:
-      LM_OK(shape(1, 1));
-      LM_CUDA(cudaMemcpy(L.w.norms + (which - MLLMB200_LM_T_NORM1), data, 4, cudaMemcpyDefault));
+      if (e->post) {
+        if (which != MLLMB200_LM_T_NORM1 && which != MLLMB200_LM_T_NORM2) return fail(e, MLLMB200_INVALID_ARG, "tensor %d: one norm per sublayer", which);
+        LM_OK(shape(1, c.width));
+        LM_OK(set_vector(e, L.w.norms + (which == MLLMB200_LM_T_NORM2 ? e->widthp : 0), data, cols));
+      } else {
+        LM_OK(shape(1, 1));
+        LM_OK(set_vector(e, L.w.norms + (which - MLLMB200_LM_T_NORM1), data, 1));
+      }
       break;
     case MLLMB200_LM_T_CONV: {
       LM_OK(shape(c.width, c.conv_taps));
@@ -427,11 +612,22 @@ int check_loaded(Engine* e) {
     const LayerState& L = e->layers[i];
     if (L.src != i) continue;
     auto bit = [](int w) { return 1u << w; };
-    unsigned need = bit(MLLMB200_LM_T_Q) | bit(MLLMB200_LM_T_K) | bit(MLLMB200_LM_T_V) | bit(MLLMB200_LM_T_O) | bit(MLLMB200_LM_T_NORM1) | bit(MLLMB200_LM_T_NORM1B);
-    if (L.d.ff) need |= bit(MLLMB200_LM_T_GATE) | bit(MLLMB200_LM_T_UP) | bit(MLLMB200_LM_T_DOWN) | bit(MLLMB200_LM_T_NORM2) | bit(MLLMB200_LM_T_NORM2B);
+    const unsigned mlp = bit(MLLMB200_LM_T_GATE) | bit(MLLMB200_LM_T_UP) | bit(MLLMB200_LM_T_DOWN);
+    unsigned need = bit(MLLMB200_LM_T_Q) | bit(MLLMB200_LM_T_O) | bit(MLLMB200_LM_T_NORM1);
+    need |= is_latent(L) ? bit(MLLMB200_LM_T_UK) | bit(MLLMB200_LM_T_UV) : bit(MLLMB200_LM_T_K) | bit(MLLMB200_LM_T_V);
+    if (owns_latent(L)) need |= bit(MLLMB200_LM_T_DKV) | bit(MLLMB200_LM_T_DKV_NORM);
+    if (!e->post) need |= bit(MLLMB200_LM_T_NORM1B);
+    if (L.d.ff) need |= bit(MLLMB200_LM_T_NORM2) | (e->post ? 0 : bit(MLLMB200_LM_T_NORM2B));
+    if (L.d.experts) {
+      need |= bit(MLLMB200_LM_T_ROUTER) | bit(MLLMB200_LM_T_ROUTER_B);
+      for (int x = 0; x < L.d.experts; ++x)
+        if (L.w.expert_loaded[x] != mlp) return fail(e, MLLMB200_INVALID_ARG, "layer %d: tensors of expert %d missing", i, x);
+    } else if (L.d.ff) {
+      need |= mlp;
+    }
     if (e->c.conv_taps) need |= bit(MLLMB200_LM_T_CONV);
     if (L.w.bias) need |= bit(MLLMB200_LM_T_REL);
-    if (!is_attn(L)) need |= bit(MLLMB200_LM_T_G) | bit(MLLMB200_LM_T_DECAY);
+    if (L.w.decay) need |= bit(MLLMB200_LM_T_G) | bit(MLLMB200_LM_T_DECAY);
     if ((L.w.loaded & need) != need) return fail(e, MLLMB200_INVALID_ARG, "layer %d: tensors missing (have %x, need %x)", i, L.w.loaded, need);
   }
   return MLLMB200_OK;
@@ -441,17 +637,14 @@ int check_loaded(Engine* e) {
 // The residual stream between sublayers: x, and the sublayer output that the next norm folds in.
 struct Stream {
   float *x, *other;
-  int planes = 0;             // of e->delta; 0 = nothing to fold in
-  size_t plane = 0;
+  Delta delta{};              // p = nullptr: nothing to fold in
   const float* gain = nullptr;
 };
 
 NormArgs norm_args(Engine* e, const StepCtx& t, const Stream& r, const float* g_pre, void* out) {
   NormArgs a{};
   a.x_in = r.x;
-  a.delta = r.planes ? e->delta : nullptr;
-  a.planes = r.planes;
-  a.plane = r.plane;
+  a.delta = r.delta;
   a.g_post = r.gain;
   a.g_pre = g_pre;
   a.eps = e->c.eps;
@@ -467,7 +660,7 @@ NormArgs norm_args(Engine* e, const StepCtx& t, const Stream& r, const float* g_
 
 int fold_norm(Engine* e, const StepCtx& t, Stream* r, const float* g_pre, LayerState* conv_layer) {
   NormArgs a = norm_args(e, t, *r, g_pre, e->h);
-  if (r->planes) a.x_out = r->other;
+  if (r->delta.p) a.x_out = r->other;
   if (conv_layer && e->c.conv_taps) {
     a.taps = e->c.conv_taps;
     a.conv_w = e->layers[conv_layer->src].w.conv;
@@ -476,8 +669,44 @@ int fold_norm(Engine* e, const StepCtx& t, Stream* r, const float* g_pre, LayerS
     if (!t.single) a.rows_per_cta = std::max(1, std::min(16, t.rows / (2 * kSms)));
   }
   LM_CUDA(launch_norm(e->stream, e->f32, a));
-  if (r->planes) std::swap(r->x, r->other);
-  r->planes = 0;
+  if (r->delta.p) std::swap(r->x, r->other);
+  r->delta = Delta{};
+  return MLLMB200_OK;
+}
+
+int linear_failed(Engine* e) { return fail(e, MLLMB200_CUDA_ERROR, "linear launch: %s", cudaGetErrorString(cudaGetLastError())); }
+
+RouterArgs router_args(Engine* e, int layer, bool gemv) {
+  const LayerState& L = e->layers[layer];
+  const Weights& w = e->layers[L.src].w;
+  RouterArgs a{};
+  a.w = w.router.w;
+  a.b = w.router_b;
+  a.experts = L.d.experts;
+  a.top = L.d.top;
+  a.ldw = w.router.k;
+  a.sel = e->route_sel;
+  a.weight = e->route_weight;
+  a.count = e->route_count + (size_t)layer * (e->n_route_count / e->c.layers);
+  a.rank = gemv ? nullptr : e->route_rank;
+  return a;
+}
+
+// x = norm(residual_scale x + sublayer), in place, and h; router: the experts of a mixture behind this norm, if it takes them.
+int post_norm(Engine* e, const StepCtx& t, Stream* r, const float* gain, const RouterArgs* router) {
+  PostNormArgs a{};
+  a.x_in = a.x_out = r->x;
+  a.delta = r->delta;
+  a.alpha = e->c.residual_scale;
+  a.gain = gain;
+  a.eps = e->c.eps;
+  a.width = e->c.width;
+  a.ldx = e->widthp;
+  a.rows = t.rows;
+  a.out = e->h;
+  if (router) a.router = *router;
+  LM_CUDA(launch_post_norm(e->stream, e->f32, a));
+  r->delta = Delta{};
   return MLLMB200_OK;
 }
 
@@ -490,9 +719,66 @@ int delta_linear(Engine* e, const StepCtx& t, const Linear& w, const ActMap& m, 
   p.ldy = e->widthp;
   p.scale = 1.0f;
   const int planes = launch_linear(e->stream, e->f32, w, m, x, t.rows, p, std::max(1, std::min(kMaxSplits, e->plane_rows / t.rows)));
-  if (planes < 1) return fail(e, MLLMB200_CUDA_ERROR, "linear launch: %s", cudaGetErrorString(cudaGetLastError()));
-  r->planes = planes;
-  r->plane = p.plane;
+  if (planes < 1) return linear_failed(e);
+  r->delta = Delta{e->delta, planes, e->widthp, p.plane, nullptr, nullptr, 1};
+  r->gain = gain;
+  return MLLMB200_OK;
+}
+
+Epi gate_epi(Engine* e, const LayerState& L, const Weights& w) {
+  Epi p{};
+  p.kind = kEpiGate;
+  p.act = e->act;
+  p.ld_act = w.down.k;
+  p.act_kind = L.d.act;
+  p.limit = L.d.ff_limit;
+  return p;
+}
+
+// A mixture of experts on e->h; `routed`: the norm before has chosen the experts.
+int moe(Engine* e, const StepCtx& t, int layer, bool routed, const float* gain, Stream* r) {
+  const LayerState& L = e->layers[layer];
+  const Weights& w = e->layers[L.src].w;
+  const int pairs = t.rows * L.d.top;
+  const bool gemv = t.rows <= kGemvRows;
+  const RouterArgs ra = router_args(e, layer, gemv);
+  if (!routed) {
+    Epi p{};
+    p.kind = kEpiPlanes;
+    p.y = e->route_logits;
+    p.ldy = pad_to(L.d.experts, 4);
+    p.plane = (size_t)t.rows * p.ldy;
+    p.scale = 1.0f;
+    const int planes = launch_linear(e->stream, e->f32, w.router, e->m_h, e->h, t.rows, p, e->route_planes);
+    if (planes < 1) return linear_failed(e);
+    LM_CUDA(launch_topk(e->stream, ra, e->route_logits, p.ldy, planes, p.plane, t.rows));
+  }
+  Groups g;
+  g.rows = pairs;
+  const void* x = e->h;
+  if (gemv) {
+    g.group_of = e->route_sel;
+    g.div = L.d.top;
+  } else {
+    LM_CUDA(launch_moe_permute(e->stream, e->f32, ra, e->h, e->widthp, t.rows, e->permuted, e->pair_row, e->moe_tiles, e->n_moe_tiles));
+    const int tile = group_tile_rows(e->f32), active = std::min(L.d.experts, pairs);
+    g.tiles = e->moe_tiles;
+    g.n_tiles = e->n_moe_tiles;
+    g.max_tiles = active + pairs / tile;
+    g.likely_tiles = active * ((pairs / active + tile - 1) / tile);
+    x = e->permuted;
+  }
+  if (launch_linear_groups(e->stream, e->f32, w.gate_up, e->m_permuted, x, g, gate_epi(e, L, w), 1) < 1) return linear_failed(e);
+  g.div = 1;
+  Epi p{};
+  p.kind = kEpiPlanes;
+  p.y = e->delta;
+  p.plane = (size_t)pairs * e->widthp;
+  p.ldy = e->widthp;
+  p.scale = 1.0f;
+  const int planes = launch_linear_groups(e->stream, e->f32, w.down, L.a_act, e->act, g, p, std::max(1, std::min(kMaxSplits, e->plane_rows / pairs)));
+  if (planes < 1) return linear_failed(e);
+  r->delta = Delta{e->delta, planes, e->widthp, p.plane, e->route_weight, gemv ? nullptr : e->pair_row, L.d.top};
   r->gain = gain;
   return MLLMB200_OK;
 }
@@ -504,7 +790,75 @@ int keep_residual(Engine* e, const StepCtx& t, int layer, const float* x) {
   return MLLMB200_OK;
 }
 
+int latent_mixer(Engine* e, const StepCtx& t, LayerState& L) {
+  const Weights& w = L.w;
+  const auto& d = L.d;
+  Epi p{};
+  p.kind = kEpiQLatent;
+  p.q = e->proj;
+  p.ldq = p.q_end = qk_cols(L);
+  p.y = e->fresh;
+  p.ldy = L.rankp;
+  if (launch_linear(e->stream, e->f32, w.in, e->m_h, e->h, t.rows, p, 1) < 1) return linear_failed(e);
+  LatentArgs a{};
+  a.heads = d.heads;
+  a.dimp = L.dimp;
+  a.vdimp = L.vdimp;
+  a.rank = d.kv_rank;
+  a.rankp = L.rankp;
+  a.max_ctx = e->c.max_ctx;
+  a.scale = d.score_scale;
+  a.eps = e->c.eps;
+  a.q = e->proj;
+  a.ldq = p.ldq;
+  a.cache = L.kc;
+  a.fresh = e->fresh;
+  a.gain = w.kv_gain;
+  a.uk_t = w.uk_t;
+  a.uv = w.uk_uv.w + (size_t)qk_cols(L) * L.rankp;
+  a.row_sp = t.row_sp;
+  a.rows = t.latent_rows;
+  a.n_rows = t.n_latent;
+  a.ctx = t.latent_ctx;
+  a.qa = e->qa;
+  a.part_o = e->lat_part;
+  a.part_ml = e->lat_ml;
+  a.lat = e->lat;
+  a.out = e->mix;
+  a.ldo = w.out.k;
+  const bool with_cache = owns_latent(L) && !t.latent_rows;  // every row attends through the latent
+  if (owns_latent(L) && !with_cache) LM_CUDA(launch_latent_cache(e->stream, e->f32, a, t.rows));
+  if (a.n_rows) LM_CUDA(launch_latent_absorbed(e->stream, e->f32, a, with_cache));
+  for (const ExpandPass& x : t.expand) {
+    Groups g;
+    g.tiles = x.rows;
+    g.max_tiles = g.likely_tiles = x.n_rows;
+    g.rows = x.total;
+    Epi kv{};
+    kv.kind = kEpiQkv;
+    kv.kc = e->ex_k;
+    kv.vc = e->ex_v;
+    kv.k_end = qk_cols(L);
+    kv.dimp = L.dimp;
+    kv.vdimp = L.vdimp;
+    kv.kv_heads = d.heads;
+    kv.max_ctx = x.total;
+    if (launch_linear_groups(e->stream, e->f32, w.uk_uv, L.a_kc, L.kc, g, kv, 1) < 1) return linear_failed(e);
+    AttnShape s{};
+    s.heads = s.kv_heads = d.heads;
+    s.dimp = L.dimp;
+    s.vdimp = L.vdimp;
+    s.slot_rows = 1;  // a tile names its sequence's first row
+    s.head_rows = x.total;
+    s.scale = d.score_scale;
+    LM_CUDA(launch_attention(e->stream, e->f32, s, e->proj, p.ldq, t.row_sp, t.rows, e->ex_k, e->ex_v, nullptr, e->mix, a.ldo, x.tiles, x.n_tiles,
+                             nullptr, 0, 0, 0, nullptr, nullptr));
+  }
+  return MLLMB200_OK;
+}
+
 int mixer(Engine* e, const StepCtx& t, LayerState& L) {
+  if (is_latent(L)) return latent_mixer(e, t, L);
   const Weights& w = e->layers[L.src].w;
   const auto& d = L.d;
   const int ldo = w.out.k;
@@ -523,13 +877,14 @@ int mixer(Engine* e, const StepCtx& t, LayerState& L) {
     p.kv_heads = d.kv_heads;
     p.max_ctx = e->c.max_ctx;
     p.row_sp = t.row_sp;
-    if (launch_linear(e->stream, e->f32, w.in, e->m_h, e->h, t.rows, p, 1) < 1) return fail(e, MLLMB200_CUDA_ERROR, "linear launch: %s", cudaGetErrorString(cudaGetLastError()));
+    if (launch_linear(e->stream, e->f32, w.in, e->m_h, e->h, t.rows, p, 1) < 1) return linear_failed(e);
     AttnShape s{};
     s.heads = d.heads;
     s.kv_heads = d.kv_heads;
     s.dimp = L.dimp;
     s.vdimp = L.vdimp;
-    s.max_ctx = e->c.max_ctx;
+    s.slot_rows = (size_t)d.kv_heads * e->c.max_ctx;
+    s.head_rows = e->c.max_ctx;
     s.sink = d.sink;
     s.has_bias = d.bias_rows > 0;
     s.bias_max = d.bias_max;
@@ -544,7 +899,7 @@ int mixer(Engine* e, const StepCtx& t, LayerState& L) {
   p.kind = kEpiPlanes;
   p.y = e->proj;
   p.ldy = 2 * (qk_cols(L) + mix_cols(L));
-  if (launch_linear(e->stream, e->f32, w.in, e->m_h, e->h, t.rows, p, 1) < 1) return fail(e, MLLMB200_CUDA_ERROR, "linear launch: %s", cudaGetErrorString(cudaGetLastError()));
+  if (launch_linear(e->stream, e->f32, w.in, e->m_h, e->h, t.rows, p, 1) < 1) return linear_failed(e);
   RetentionArgs a{};
   a.qkvg = e->proj;
   a.ld = p.ldy;
@@ -573,10 +928,36 @@ int mixer(Engine* e, const StepCtx& t, LayerState& L) {
   return MLLMB200_OK;
 }
 
+// Layers with the norms behind the residual sum; the sublayers read x itself.
+int forward_post(Engine* e, const StepCtx& t, Stream* r) {
+  for (int l = 0; l < e->c.layers; ++l) {
+    LayerState& L = e->layers[l];
+    const Weights& w = e->layers[L.src].w;
+    const bool routed = L.d.experts && fused_router(t.rows);
+    LM_OK(mixer(e, t, L));
+    LM_OK(delta_linear(e, t, w.out, L.a_mix, e->mix, nullptr, r));
+    const RouterArgs ra = router_args(e, l, t.rows <= kGemvRows);
+    LM_OK(post_norm(e, t, r, w.norms, routed ? &ra : nullptr));
+    if (L.d.ff) {
+      if (L.d.experts) {
+        LM_OK(moe(e, t, l, routed, nullptr, r));
+      } else {
+        if (launch_linear(e->stream, e->f32, w.gate_up, e->m_h, e->h, t.rows, gate_epi(e, L, w), 1) < 1) return linear_failed(e);
+        LM_OK(delta_linear(e, t, w.down, L.a_act, e->act, nullptr, r));
+      }
+      LM_OK(post_norm(e, t, r, w.norms + e->widthp, nullptr));
+    }
+    LM_OK(keep_residual(e, t, l, r->x));
+  }
+  return MLLMB200_OK;
+}
+
 int forward(Engine* e, const StepCtx& t, Stream* r) {
   r->x = e->xa;
   r->other = e->xb;
-  LM_CUDA(launch_embed(e->stream, t.tokens, e->embed, e->c.width, e->widthp, t.rows, r->x));
+  LM_CUDA(launch_embed(e->stream, e->f32, t.tokens, e->embed, e->c.width, e->widthp, t.rows, r->x, e->post ? e->h : nullptr, e->route_count,
+                       e->n_route_count));
+  if (e->post) return forward_post(e, t, r);
   for (int l = 0; l < e->c.layers; ++l) {
     LayerState& L = e->layers[l];
     const Weights& w = e->layers[L.src].w;
@@ -586,12 +967,11 @@ int forward(Engine* e, const StepCtx& t, Stream* r) {
     LM_OK(delta_linear(e, t, w.out, L.a_mix, e->mix, w.norms + 1, r));
     if (!L.d.ff) continue;
     LM_OK(fold_norm(e, t, r, w.norms + 2, nullptr));
-    Epi p{};
-    p.kind = kEpiGate;
-    p.act = e->act;
-    p.ld_act = w.down.k;
-    p.limit = L.d.ff_limit;
-    if (launch_linear(e->stream, e->f32, w.gate_up, e->m_h, e->h, t.rows, p, 1) < 1) return fail(e, MLLMB200_CUDA_ERROR, "linear launch: %s", cudaGetErrorString(cudaGetLastError()));
+    if (L.d.experts) {
+      LM_OK(moe(e, t, l, false, w.norms + 3, r));
+      continue;
+    }
+    if (launch_linear(e->stream, e->f32, w.gate_up, e->m_h, e->h, t.rows, gate_epi(e, L, w), 1) < 1) return linear_failed(e);
     LM_OK(delta_linear(e, t, w.down, L.a_act, e->act, w.norms + 3, r));
   }
   if (e->keep) {
@@ -605,16 +985,30 @@ int forward(Engine* e, const StepCtx& t, Stream* r) {
 
 // Logits of n <= logit_rows rows named by `gather` (device) into e->logits.
 int logits_of(Engine* e, const StepCtx& t, const Stream& r, const int* gather, int n) {
-  NormArgs a = norm_args(e, t, r, e->final_gain, e->hf);
-  a.gather = gather;
-  a.rows = n;
-  LM_CUDA(launch_norm(e->stream, e->f32, a));
+  if (e->post) {
+    PostNormArgs a{};
+    a.x_in = r.x;
+    a.alpha = 1.0f;
+    a.gain = e->final_gain;
+    a.eps = e->c.eps;
+    a.width = e->c.width;
+    a.ldx = e->widthp;
+    a.rows = n;
+    a.out = e->hf;
+    a.gather = gather;
+    LM_CUDA(launch_post_norm(e->stream, e->f32, a));
+  } else {
+    NormArgs a = norm_args(e, t, r, e->final_gain, e->hf);
+    a.gather = gather;
+    a.rows = n;
+    LM_CUDA(launch_norm(e->stream, e->f32, a));
+  }
   Epi p{};
   p.kind = kEpiPlanes;
   p.y = e->logits;
   p.ldy = e->c.vocab;
   p.scale = e->c.logit_scale;
-  if (launch_linear(e->stream, e->f32, e->head, e->m_hf, e->hf, n, p, 1) < 1) return fail(e, MLLMB200_CUDA_ERROR, "linear launch: %s", cudaGetErrorString(cudaGetLastError()));
+  if (launch_linear(e->stream, e->f32, e->head, e->m_hf, e->hf, n, p, 1) < 1) return linear_failed(e);
   return MLLMB200_OK;
 }
 
@@ -718,8 +1112,36 @@ int step(Engine* e, int n_entries, const int* slots, const int* counts, const in
       }
     }
   }
-  for (auto& g : tiles)  // tiles with the longest causal range first
-    std::stable_sort(g.second.begin(), g.second.end(), [](const int4& a, const int4& b) { return a.w + a.y > b.w + b.y; });
+  auto longest_first = [](std::vector<int4>* v) {  // by causal range
+    std::stable_sort(v->begin(), v->end(), [](const int4& a, const int4& b) { return a.w + a.y > b.w + b.y; });
+  };
+  for (auto& g : tiles) longest_first(&g.second);
+
+  struct Pass {
+    std::vector<int4> rows, tiles;
+    int total = 0;
+  };
+  std::vector<Pass> passes;
+  std::vector<int> latent_rows;
+  int latent_ctx = 1;
+  bool all_latent = true;
+  if (e->latent)
+    for (const Entry& en : entries) {
+      const int ctx = en.pos0 + en.count;
+      if (e->f32 || en.count <= kAbsorbMax) {
+        for (int j = 0; j < en.count; ++j) latent_rows.push_back(en.row0 + j);
+        latent_ctx = std::max(latent_ctx, ctx);
+        continue;
+      }
+      all_latent = false;
+      if (passes.empty() || passes.back().total + ctx > e->expand_cap) passes.emplace_back();
+      Pass& ps = passes.back();
+      const int first = ps.total, cache0 = en.slot * c.max_ctx, tile = group_tile_rows(false), toks = attention_tile_rows();
+      for (int j = 0; j < ctx; j += tile) ps.rows.push_back(make_int4(0, cache0 + j, std::min(tile, ctx - j), first + j));
+      for (int j = 0; j < en.count; j += toks) ps.tiles.push_back(make_int4(en.row0 + j, std::min(toks, en.count - j), first, en.pos0 + j));
+      ps.total += ctx;
+    }
+  for (auto& ps : passes) longest_first(&ps.tiles);
 
   MetaBuilder m(e->meta);
   const size_t o_tok = m.add(tokens, rows), o_sp = m.add(row_sp.data(), 2 * (size_t)rows), o_re = m.add(row_entry.data(), rows);
@@ -729,6 +1151,12 @@ int step(Engine* e, int n_entries, const int* slots, const int* counts, const in
   const size_t o_sl = m.add(slots, n_entries), o_want = m.add(want, n_want);
   std::map<int, size_t> o_tiles;
   for (auto& g : tiles) o_tiles[g.first] = m.add(g.second.data(), 4 * g.second.size());
+  const size_t o_lat = m.add(latent_rows.data(), latent_rows.size());
+  std::vector<std::pair<size_t, size_t>> o_pass;
+  for (auto& ps : passes) {
+    const size_t o_rows = m.add(ps.rows.data(), 4 * ps.rows.size());
+    o_pass.push_back({o_rows, m.add(ps.tiles.data(), 4 * ps.tiles.size())});
+  }
   LM_OK(upload_meta(e));
 
   const int* d = e->meta_d;
@@ -748,6 +1176,13 @@ int step(Engine* e, int n_entries, const int* slots, const int* counts, const in
   t.chunk = decode_chunk(t.n_single, max_single + 1);
   t.splits = max_single / t.chunk + 1;
   for (auto& g : tiles) t.tiles[g.first] = {reinterpret_cast<const int4*>(d + o_tiles[g.first]), (int)g.second.size()};
+
+  t.latent_rows = all_latent ? nullptr : d + o_lat;
+  t.n_latent = (int)latent_rows.size();
+  t.latent_ctx = latent_ctx;
+  for (size_t i = 0; i < passes.size(); ++i)
+    t.expand.push_back({reinterpret_cast<const int4*>(d + o_pass[i].first), reinterpret_cast<const int4*>(d + o_pass[i].second),
+                        (int)passes[i].rows.size(), (int)passes[i].tiles.size(), passes[i].total});
 
   const long long before = g_launches;
   Stream r{};
@@ -784,6 +1219,8 @@ int enqueue_decode(Engine* e, int count, int chunk, int splits) {
   t.single = true;
   t.chunk = chunk;
   t.splits = splits;
+  t.n_latent = count;
+  t.latent_ctx = std::min(chunk * splits, e->c.max_ctx);
   LM_CUDA(launch_decode_prep(e->stream, count, e->d_slots, e->d_pos, e->d_token, e->d_tail, e->d_row_sp, e->d_row_token, e->d_entries, e->d_row_entry));
   Stream r{};
   LM_OK(forward(e, t, &r));
@@ -887,6 +1324,10 @@ void mllmb200_lm_destroy(void* handle) {
 int mllmb200_lm_set_tensor(void* handle, int layer, int which, const void* data, int rows, int cols) {
   if (!handle || !data) return MLLMB200_INVALID_ARG;
   return set_tensor(from(handle), layer, which, data, rows, cols);
+}
+int mllmb200_lm_set_expert(void* handle, int layer, int expert, int which, const void* data, int rows, int cols) {
+  if (!handle || !data) return MLLMB200_INVALID_ARG;
+  return set_expert(from(handle), layer, expert, which, data, rows, cols);
 }
 int mllmb200_lm_step(void* handle, int entries, const int* slots, const int* counts, const int* tokens, int n_want, const int* want,
                      float* logits_out, int sample) {

@@ -4,6 +4,8 @@
 //     thread issues tcgen05.mma, the accumulators sit in tensor memory - two of them, so that a persistent CTA's
 //     epilogue of one tile overlaps the next tile's K loop.
 //   * lm_gemm_f32_kernel: fp32 activations and fp32 FMAs (the 32-bit mode of the engine), more than four rows.
+// Each also comes in a form for groups of rows with a weight each (experts), or scattered runs of rows of x: the GEMMs
+// then take a table of row tiles, whose length may be known on the device only.
 // The epilogue scatters queries, keys and values (keys and values go straight into the caches), applies the gated
 // clamped activation to interleaved gate/up columns, or leaves fp32 sums - in several planes when K is split, which
 // the consumer (a norm) adds in plane order.
@@ -27,9 +29,11 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
-__device__ __forceinline__ float gated(float g, float u, float limit) {
-  g = fminf(g, limit);
-  u = fminf(fmaxf(u, -limit), limit);
+__device__ __forceinline__ float gated(const Epi& e, float g, float u) {
+  if (e.act_kind == MLLMB200_LM_ACT_GELU) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+  if (e.act_kind == MLLMB200_LM_ACT_SILU) return g / (1.0f + expf(-g)) * u;
+  g = fminf(g, e.limit);
+  u = fminf(fmaxf(u, -e.limit), e.limit);
   return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
 }
 
@@ -37,7 +41,7 @@ __device__ __forceinline__ float gated(float g, float u, float limit) {
 template <class T>
 __device__ __forceinline__ T* qkv_ptr(const Epi& e, int m, int n) {
   if (n < e.q_end) return static_cast<T*>(e.q) + (size_t)m * e.ldq + n;
-  const int2 sp = e.row_sp[m];
+  const int2 sp = e.row_sp ? e.row_sp[m] : make_int2(0, m);
   const bool is_k = n < e.k_end;
   const int d = is_k ? e.dimp : e.vdimp;
   const int c = n - (is_k ? e.q_end : e.k_end), g = c / d;
@@ -52,12 +56,16 @@ __device__ __forceinline__ void store2(const Epi& e, int m, int n, int N, float 
     float* y = e.y + (size_t)split * e.plane + (size_t)m * e.ldy + n;
     y[0] = v0 * e.scale;
     if (n + 1 < N) y[1] = v1 * e.scale;
-  } else if (e.kind == kEpiQkv) {
+  } else if (e.kind == kEpiQLatent && n >= e.q_end) {
+    float* y = e.y + (size_t)m * e.ldy + (n - e.q_end);
+    y[0] = v0;
+    y[1] = v1;
+  } else if (e.kind != kEpiGate) {
     T* p = qkv_ptr<T>(e, m, n);
     p[0] = from_f32<T>(v0);
     p[1] = from_f32<T>(v1);
   } else {
-    static_cast<T*>(e.act)[(size_t)m * e.ld_act + (n >> 1)] = from_f32<T>(gated(v0, v1, e.limit));
+    static_cast<T*>(e.act)[(size_t)m * e.ld_act + (n >> 1)] = from_f32<T>(gated(e, v0, v1));
   }
 }
 
@@ -80,14 +88,18 @@ __device__ __forceinline__ void store16(const Epi& e, int m, int n, int N, const
       for (int i = 0; i < 16; ++i)
         if (n + i < N) y[i] = v[i] * e.scale;
     }
-  } else if (e.kind == kEpiQkv) {  // head sizes are multiples of 16: the chunk lies in one head
+  } else if (e.kind == kEpiQLatent && n >= e.q_end) {
+    float4* y = reinterpret_cast<float4*>(e.y + (size_t)m * e.ldy + (n - e.q_end));
+#pragma unroll
+    for (int i = 0; i < 4; ++i) y[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+  } else if (e.kind != kEpiGate) {  // head sizes are multiples of 16: the chunk lies in one head
     uint4* p = reinterpret_cast<uint4*>(qkv_ptr<__nv_bfloat16>(e, m, n));
     p[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
     p[1] = make_uint4(pack_bf16(v[8], v[9]), pack_bf16(v[10], v[11]), pack_bf16(v[12], v[13]), pack_bf16(v[14], v[15]));
-  } else {  // pairs past N are zero rows of the weight tile: they write zeros into the padding of the row
+  } else {  // pairs past N write zeros into the padding of the row
     float a[8];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] = gated(v[2 * i], v[2 * i + 1], e.limit);
+    for (int i = 0; i < 8; ++i) a[i] = n + 2 * i < N ? gated(e, v[2 * i], v[2 * i + 1]) : 0.0f;
     *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(e.act) + (size_t)m * e.ld_act + (n >> 1)) =
         make_uint4(pack_bf16(a[0], a[1]), pack_bf16(a[2], a[3]), pack_bf16(a[4], a[5]), pack_bf16(a[6], a[7]));
   }
@@ -110,10 +122,12 @@ __device__ __forceinline__ void load8(const float* p, float (&f)[8]) {
   f[0] = a.x, f[1] = a.y, f[2] = a.z, f[3] = a.w, f[4] = b.x, f[5] = b.y, f[6] = b.z, f[7] = b.w;
 }
 
-// A group of 2^ks_log2 warps owns output columns (2 p, 2 p + 1); its warps split K.
+// A group of 2^ks_log2 warps owns output columns (2 p, 2 p + 1); its warps split K.  With group_of, CTA row y makes result
+// row y from row y / div of x and weight group group_of[y].
 template <class T, int MT>
 __global__ void __launch_bounds__(kGemvThreads) lm_gemv_kernel(const T* __restrict__ x, const __nv_bfloat16* __restrict__ w,
-                                                               int N, int K, int ks_log2, Epi e) {
+                                                               int N, int K, int ks_log2, const int* __restrict__ group_of, int div,
+                                                               Epi e) {
   extern __shared__ __align__(16) uint8_t gemv_smem[];
   __shared__ float red[kGemvWarps][2 * MT];
   T* xs = reinterpret_cast<T*>(gemv_smem);
@@ -135,8 +149,15 @@ __global__ void __launch_bounds__(kGemvThreads) lm_gemv_kernel(const T* __restri
     }
   };
   pdl_launch_dependents();
-  fetch(i0);  // the weights do not depend on the previous kernel
+  if (!group_of) fetch(i0);  // the weights do not depend on the previous kernel
   pdl_wait_prior();
+  const int m0 = group_of ? blockIdx.y : 0;
+  if (group_of) {
+    w0 += (size_t)group_of[m0] * N * K;
+    w1 = w0 + K;
+    x += (size_t)(m0 / div) * K;
+    fetch(i0);
+  }
   constexpr int kVec = 16 / sizeof(T);
   for (int i = tid; i < MT * K / kVec; i += kGemvThreads) reinterpret_cast<uint4*>(xs)[i] = reinterpret_cast<const uint4*>(x)[i];
   __syncthreads();
@@ -182,7 +203,7 @@ __global__ void __launch_bounds__(kGemvThreads) lm_gemv_kernel(const T* __restri
       v0 += red[warp + j][lane];
       v1 += red[warp + j][MT + lane];
     }
-    store2<T>(e, lane, n0, N, v0, v1, 0);
+    store2<T>(e, m0 + lane, n0, N, v0, v1, 0);
   }
 }
 
@@ -190,12 +211,21 @@ __global__ void __launch_bounds__(kGemvThreads) lm_gemv_kernel(const T* __restri
 constexpr int kF32Tile = 64, kF32K = 32;
 
 __global__ void __launch_bounds__(256) lm_gemm_f32_kernel(const float* __restrict__ x, const __nv_bfloat16* __restrict__ w, int M,
-                                                          int N, int K, Epi e) {
+                                                          int N, int K, const int4* __restrict__ tiles, const int* __restrict__ n_tiles,
+                                                          Epi e) {
   __shared__ __align__(16) float xs[kF32K][kF32Tile + 4], ws[kF32K][kF32Tile + 4];
   pdl_launch_dependents();
   pdl_wait_prior();
   const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
-  const int m0 = blockIdx.y * kF32Tile, n0 = blockIdx.x * kF32Tile;
+  int m0 = blockIdx.y * kF32Tile, out0 = 0;
+  const int n0 = blockIdx.x * kF32Tile;
+  if (tiles) {
+    if (n_tiles && (int)blockIdx.y >= *n_tiles) return;
+    const int4 t = tiles[blockIdx.y];
+    w += (size_t)t.x * N * K;
+    x += (size_t)t.y * K;
+    M = t.z, out0 = t.w, m0 = 0;
+  }
   float acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += kF32K) {
     for (int i = tid; i < kF32Tile * kF32K / 4; i += 256) {
@@ -230,7 +260,7 @@ __global__ void __launch_bounds__(256) lm_gemm_f32_kernel(const float* __restric
 #pragma unroll
     for (int j = 0; j < 4; j += 2) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) store2<float>(e, m, n, N, acc[i][j], acc[i][j + 1], 0);
+      if (n < N) store2<float>(e, out0 + m, n, N, acc[i][j], acc[i][j + 1], 0);
     }
   }
 }
@@ -260,10 +290,14 @@ __device__ __forceinline__ uint64_t swizzled_desc(uint32_t addr) {
 }
 
 // Work items are (K split, weight tile, row tile), row tiles fastest; CTA c takes items c, c + gridDim.x, ...
-template <int BN>
+// GROUPED: the row tiles are those of `tiles`; whole tiles are copied through amap (boxes of 128 rows), the others through
+// amap16 (16 rows).  Weight tiles and boxes may reach into the next group: those sums are not stored.
+template <int BN, bool GROUPED>
 __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_constant__ CUtensorMap amap,
+                                                                   const __grid_constant__ CUtensorMap amap16,
                                                                    const __grid_constant__ CUtensorMap wmap, int a_box, int M, int N,
-                                                                   int K, int splits, Epi e) {
+                                                                   int K, int splits, const int4* __restrict__ tiles,
+                                                                   const int* __restrict__ n_tiles, int max_tiles, Epi e) {
   using S = TcShape<BN>;
   extern __shared__ uint8_t tc_smem_raw[];
   __shared__ uint64_t full[S::kStages], empty[S::kStages], acc_full[2], acc_empty[2];
@@ -271,9 +305,13 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
   __shared__ volatile int gave_up;
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(tc_smem_raw) + 1023) & ~(uintptr_t)1023);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int mt = (M + kTileM - 1) / kTileM, nt = (N + BN - 1) / BN, kt = K / kTileK;
-  const int items = mt * nt * splits;
-  const int a_rows = M >= kTileM ? kTileM : (M + 15) / 16 * 16;  // rows of x that are loaded at all
+  int mt = (M + kTileM - 1) / kTileM;
+  const int nt = (N + BN - 1) / BN, kt = K / kTileK;
+  int a_rows = M >= kTileM ? kTileM : (M + 15) / 16 * 16;  // rows of x that are loaded at all
+  auto grouped_start = [&]() {
+    pdl_wait_prior();
+    mt = n_tiles ? min(*n_tiles, max_tiles) : max_tiles;
+  };
   constexpr int kWBox = BN < 128 ? 32 : 128;
   if (tid == 0) {
     for (int i = 0; i < S::kStages; ++i) mbar_init(&full[i], 1), mbar_init(&empty[i], 1);
@@ -299,20 +337,30 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
       int it = 0, ahead = 0;
       bool ok = true;
       auto stage = [&](int i) { return smem + (size_t)(i % S::kStages) * S::kStageBytes; };
-      auto load_w = [&](int i, int k, int n0) {
+      auto load_w = [&](int i, int k, int w_row) {
         mbar_arrive_expect_tx(&full[i % S::kStages], (uint32_t)(a_rows + BN) * kTileK * 2);
         for (int b = 0; b < BN; b += kWBox)
-          tma_load_2d(stage(i) + kABytes + b * kTileK * 2, &wmap, k * kTileK, n0 + b, &full[i % S::kStages]);
+          tma_load_2d(stage(i) + kABytes + b * kTileK * 2, &wmap, k * kTileK, w_row + b, &full[i % S::kStages]);
       };
-      {  // the weights do not depend on the previous kernel, the activations do: fill the ring with weights first
+      if (GROUPED) {
+        grouped_start();
+      } else {  // the weights do not depend on the previous kernel, the activations do: fill the ring with weights first
         const int item = blockIdx.x;
         int k0, k1;
         k_range(item / (mt * nt), k0, k1);
         for (; ahead < S::kStages && ahead < k1 - k0; ++ahead) load_w(ahead, k0 + ahead, (item / mt % nt) * BN);
         pdl_wait_prior();
       }
-      for (int item = blockIdx.x; item < items && ok; item += gridDim.x) {
-        const int m0 = (item % mt) * kTileM, n0 = (item / mt % nt) * BN;
+      for (int item = blockIdx.x; item < mt * nt * splits && ok; item += gridDim.x) {
+        int x_row = (item % mt) * kTileM, w_row = (item / mt % nt) * BN;
+        if (GROUPED) {
+          const int4 t = tiles[item % mt];
+          x_row = t.y;
+          w_row += t.x * N;
+          a_box = t.z > kTileM - 16 ? kTileM : 16;
+          a_rows = (t.z + 15) / 16 * 16;
+        }
+        const CUtensorMap* am = !GROUPED || a_box == kTileM ? &amap : &amap16;
         int k0, k1;
         k_range(item / (mt * nt), k0, k1);
         for (int k = k0; k < k1; ++k, ++it) {
@@ -321,8 +369,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
             ok = false;
             break;
           }
-          if (it >= ahead) load_w(it, k, n0);
-          for (int b = 0; b < a_rows; b += a_box) tma_load_2d(stage(it) + b * kTileK * 2, &amap, k * kTileK, m0 + b, &full[st]);
+          if (it >= ahead) load_w(it, k, w_row);
+          for (int b = 0; b < a_rows; b += a_box) tma_load_2d(stage(it) + b * kTileK * 2, am, k * kTileK, x_row + b, &full[st]);
         }
       }
       if (!ok) gave_up = 1;
@@ -335,7 +383,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
     const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kTileM >> 4) << 24);
     int it = 0, t = 0;
     bool ok = true;
-    for (int item = blockIdx.x; item < items && ok; item += gridDim.x, ++t) {
+    if (GROUPED) grouped_start();
+    for (int item = blockIdx.x; item < mt * nt * splits && ok; item += gridDim.x, ++t) {
       int k0, k1;
       k_range(item / (mt * nt), k0, k1);
       const int buf = t & 1;
@@ -363,19 +412,26 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
     }
     if (!ok) gave_up = 1;
   } else {
-    pdl_wait_prior();  // outputs may still be read by the kernel before
+    if (GROUPED) grouped_start();
+    else pdl_wait_prior();  // outputs may still be read by the kernel before
     const int quarter = warp & 3;
     int t = 0;
-    for (int item = blockIdx.x; item < items; item += gridDim.x, ++t) {
+    for (int item = blockIdx.x; item < mt * nt * splits; item += gridDim.x, ++t) {
       const int buf = t & 1;
       if (gave_up || !mbar_wait_bounded(&acc_full[buf], (t >> 1) & 1)) {
         gave_up = 1;
         break;
       }
       tc_fence_after();
-      const int m0 = (item % mt) * kTileM, n0 = (item / mt % nt) * BN, split = item / (mt * nt);
+      const int n0 = (item / mt % nt) * BN, split = item / (mt * nt);
+      int m0 = (item % mt) * kTileM, m_end = M;
+      if (GROUPED) {
+        const int4 tile = tiles[item % mt];
+        m0 = tile.w;
+        m_end = tile.w + tile.z;
+      }
       const int m = m0 + quarter * 32 + lane;
-      if (m0 + quarter * 32 < M) {
+      if (m0 + quarter * 32 < m_end) {
         const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16) + buf * BN;
 #pragma unroll
         for (int c = 0; c < BN; c += 32) {
@@ -385,7 +441,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
           tmem_ld16(base + c + 16, r1);
           tmem_ld_wait();
           float v[16];
-          if (m < M) {
+          if (m < m_end) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r0[i]);
             store16(e, m, n0 + c, N, v, split);
@@ -419,6 +475,15 @@ __global__ void lm_pack_rows_kernel(const __nv_bfloat16* __restrict__ src, int n
   }
 }
 
+__global__ void lm_pack_heads_transposed_kernel(const __nv_bfloat16* __restrict__ src, int heads, int dim, int rank,
+                                                __nv_bfloat16* __restrict__ dst, int rankp, int dimp) {
+  for (int r = blockIdx.x; r < heads * rank; r += gridDim.x) {
+    const int h = r / rank, c = r - h * rank;
+    for (int d = threadIdx.x; d < dim; d += blockDim.x)
+      dst[((size_t)h * rankp + c) * dimp + d] = src[((size_t)h * dim + d) * rank + c];
+  }
+}
+
 using EncodeFn = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
                               const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                               CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -440,9 +505,8 @@ int encode(CUtensorMap* map, const void* base, int rows, int k, int box_rows) {
 }
 
 // Tile width and K splits with the smallest estimated time: waves x (K tiles x cycles per K tile + fixed cost).
-void choose_tile(int M, int N, int K, int max_splits, int* bn_out, int* splits_out) {
-  const int mt = (M + kTileM - 1) / kTileM, kt = K / kTileK;
-  const int a_rows = M >= kTileM ? kTileM : pad_to(M, 16);
+void choose_tile(int M, int mt, int a_rows, int N, int K, int max_splits, int* bn_out, int* splits_out) {
+  const int kt = K / kTileK;
   double best = 1e30;
   for (int bn : {256, 128, 64, 32}) {
     const int nt = (N + bn - 1) / bn;
@@ -458,29 +522,33 @@ void choose_tile(int M, int N, int K, int max_splits, int* bn_out, int* splits_o
 }
 
 template <int BN>
-cudaError_t launch_tc(cudaStream_t s, const Linear& w, const ActMap& am, int M, int splits, const Epi& e) {
-  const int mt = (M + kTileM - 1) / kTileM, nt = (w.n + BN - 1) / BN;
-  const int grid = std::min(mt * nt * splits, kSms);
-  return launch_pdl(lm_gemm_tc_kernel<BN>, dim3(grid), dim3(kTcThreads), TcShape<BN>::kSmem, s, M >= kTileM ? am.map128 : am.map16,
-                    BN < 128 ? w.map32 : w.map128, M >= kTileM ? 128 : 16, M, w.n, w.k, splits, e);
+cudaError_t launch_tc(cudaStream_t s, const Linear& w, const ActMap& am, int M, int splits, const Groups* g, const Epi& e) {
+  const int nt = (w.n + BN - 1) / BN;
+  const CUtensorMap& wmap = BN < 128 ? w.map32 : w.map128;
+  if (g)
+    return launch_pdl(lm_gemm_tc_kernel<BN, true>, dim3(std::min(g->max_tiles * nt * splits, kSms)), dim3(kTcThreads), TcShape<BN>::kSmem, s,
+                      am.map128, am.map16, wmap, 128, M, w.n, w.k, splits, g->tiles, g->n_tiles, g->max_tiles, e);
+  const int mt = (M + kTileM - 1) / kTileM;
+  return launch_pdl(lm_gemm_tc_kernel<BN, false>, dim3(std::min(mt * nt * splits, kSms)), dim3(kTcThreads), TcShape<BN>::kSmem, s,
+                    M >= kTileM ? am.map128 : am.map16, am.map16, wmap, M >= kTileM ? 128 : 16, M, w.n, w.k, splits, nullptr, nullptr, 0, e);
 }
 
 template <class T, int MT>
-cudaError_t launch_gemv_mt(cudaStream_t s, const Linear& w, const void* x, const Epi& e) {
+cudaError_t launch_gemv_mt(cudaStream_t s, const Linear& w, const void* x, const Groups* g, const Epi& e) {
   int ks = 0;
-  const int pairs = (w.n + 1) / 2;
-  while (ks < 3 && ((long long)pairs << ks) / kGemvWarps < 2 * kSms && (w.k >> (8 + ks)) >= 2) ++ks;
+  const int pairs = (w.n + 1) / 2, ys = g ? g->rows : 1;
+  while (ks < 3 && ((long long)pairs * ys << ks) / kGemvWarps < 2 * kSms && (w.k >> (8 + ks)) >= 2) ++ks;
   const int per_cta = kGemvWarps >> ks;
-  return launch_pdl(lm_gemv_kernel<T, MT>, dim3((pairs + per_cta - 1) / per_cta), dim3(kGemvThreads), (size_t)MT * w.k * sizeof(T), s,
-                    static_cast<const T*>(x), w.w, w.n, w.k, ks, e);
+  return launch_pdl(lm_gemv_kernel<T, MT>, dim3((pairs + per_cta - 1) / per_cta, ys), dim3(kGemvThreads), (size_t)MT * w.k * sizeof(T), s,
+                    static_cast<const T*>(x), w.w, w.n, w.k, ks, g ? g->group_of : nullptr, g ? g->div : 1, e);
 }
 template <class T>
 cudaError_t launch_gemv(cudaStream_t s, const Linear& w, const void* x, int M, const Epi& e) {
   switch (M) {
-    case 1: return launch_gemv_mt<T, 1>(s, w, x, e);
-    case 2: return launch_gemv_mt<T, 2>(s, w, x, e);
-    case 3: return launch_gemv_mt<T, 3>(s, w, x, e);
-    default: return launch_gemv_mt<T, 4>(s, w, x, e);
+    case 1: return launch_gemv_mt<T, 1>(s, w, x, nullptr, e);
+    case 2: return launch_gemv_mt<T, 2>(s, w, x, nullptr, e);
+    case 3: return launch_gemv_mt<T, 3>(s, w, x, nullptr, e);
+    default: return launch_gemv_mt<T, 4>(s, w, x, nullptr, e);
   }
 }
 constexpr size_t kGemvSmemMax = 200 * 1024;
@@ -500,10 +568,18 @@ cudaError_t configure_gemv() {
 }  // namespace
 
 cudaError_t linear_configure() {
-  cudaError_t r = cudaFuncSetAttribute(lm_gemm_tc_kernel<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcShape<256>::kSmem);
-  if (r == cudaSuccess) r = cudaFuncSetAttribute(lm_gemm_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcShape<128>::kSmem);
-  if (r == cudaSuccess) r = cudaFuncSetAttribute(lm_gemm_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcShape<64>::kSmem);
-  if (r == cudaSuccess) r = cudaFuncSetAttribute(lm_gemm_tc_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcShape<32>::kSmem);
+  cudaError_t r = cudaSuccess;
+  auto set = [&](auto f, int bytes) {
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
+  };
+  set(lm_gemm_tc_kernel<256, false>, TcShape<256>::kSmem);
+  set(lm_gemm_tc_kernel<128, false>, TcShape<128>::kSmem);
+  set(lm_gemm_tc_kernel<64, false>, TcShape<64>::kSmem);
+  set(lm_gemm_tc_kernel<32, false>, TcShape<32>::kSmem);
+  set(lm_gemm_tc_kernel<256, true>, TcShape<256>::kSmem);
+  set(lm_gemm_tc_kernel<128, true>, TcShape<128>::kSmem);
+  set(lm_gemm_tc_kernel<64, true>, TcShape<64>::kSmem);
+  set(lm_gemm_tc_kernel<32, true>, TcShape<32>::kSmem);
   if (r == cudaSuccess) r = configure_gemv<float>();
   if (r == cudaSuccess) r = configure_gemv<__nv_bfloat16>();
   return r;
@@ -514,30 +590,60 @@ int make_act_map(ActMap* m, const void* buf, int rows, int k) {
   return st != MLLMB200_OK ? st : encode(&m->map128, buf, rows, k, 128);
 }
 int make_linear_maps(Linear* l) {
-  const int st = encode(&l->map32, l->w, l->n, l->k, 32);
-  return st != MLLMB200_OK ? st : encode(&l->map128, l->w, l->n, l->k, 128);
+  const int st = encode(&l->map32, l->w, l->n * l->groups, l->k, 32);
+  return st != MLLMB200_OK ? st : encode(&l->map128, l->w, l->n * l->groups, l->k, 128);
 }
+
+namespace {
+cudaError_t launch_tc_any(cudaStream_t s, int bn, const Linear& w, const ActMap& am, int M, int splits, const Groups* g, const Epi& e) {
+  return bn == 256   ? launch_tc<256>(s, w, am, M, splits, g, e)
+         : bn == 128 ? launch_tc<128>(s, w, am, M, splits, g, e)
+         : bn == 64  ? launch_tc<64>(s, w, am, M, splits, g, e)
+                     : launch_tc<32>(s, w, am, M, splits, g, e);
+}
+}  // namespace
+
+int group_tile_rows(bool f32) { return f32 ? kF32Tile : kTileM; }
 
 int launch_linear(cudaStream_t s, bool f32, const Linear& w, const ActMap& am, const void* x, int M, const Epi& e, int max_splits) {
   cudaError_t r;
   int splits = 1;
   const size_t elt = f32 ? 4 : 2;
-  if (M <= 4 && (size_t)M * w.k * elt <= kGemvSmemMax) {
+  if (M <= kGemvRows && (size_t)M * w.k * elt <= kGemvSmemMax) {
     r = f32 ? launch_gemv<float>(s, w, x, M, e) : launch_gemv<__nv_bfloat16>(s, w, x, M, e);
   } else if (f32) {
     r = launch_pdl(lm_gemm_f32_kernel, dim3((w.n + kF32Tile - 1) / kF32Tile, (M + kF32Tile - 1) / kF32Tile), dim3(256), 0, s,
-                   static_cast<const float*>(x), w.w, M, w.n, w.k, e);
+                   static_cast<const float*>(x), w.w, M, w.n, w.k, nullptr, nullptr, e);
   } else {
     int bn = 32;
-    choose_tile(M, w.n, w.k, e.kind == kEpiPlanes ? max_splits : 1, &bn, &splits);
-    r = bn == 256   ? launch_tc<256>(s, w, am, M, splits, e)
-        : bn == 128 ? launch_tc<128>(s, w, am, M, splits, e)
-        : bn == 64  ? launch_tc<64>(s, w, am, M, splits, e)
-                    : launch_tc<32>(s, w, am, M, splits, e);
+    choose_tile(M, (M + kTileM - 1) / kTileM, M >= kTileM ? kTileM : pad_to(M, 16), w.n, w.k, e.kind == kEpiPlanes ? max_splits : 1, &bn, &splits);
+    r = launch_tc_any(s, bn, w, am, M, splits, nullptr, e);
   }
   return r == cudaSuccess ? splits : -1;
 }
 
+int launch_linear_groups(cudaStream_t s, bool f32, const Linear& w, const ActMap& am, const void* x, const Groups& g, const Epi& e, int max_splits) {
+  cudaError_t r;
+  int splits = 1;
+  if (g.group_of) {
+    r = f32 ? launch_gemv_mt<float, 1>(s, w, x, &g, e) : launch_gemv_mt<__nv_bfloat16, 1>(s, w, x, &g, e);
+  } else if (f32) {
+    r = launch_pdl(lm_gemm_f32_kernel, dim3((w.n + kF32Tile - 1) / kF32Tile, g.max_tiles), dim3(256), 0, s, static_cast<const float*>(x), w.w, 0,
+                   w.n, w.k, g.tiles, g.n_tiles, e);
+  } else {
+    int bn = 32;
+    const int per = (g.rows + g.likely_tiles - 1) / g.likely_tiles;
+    choose_tile(g.rows, g.likely_tiles, std::min(kTileM, pad_to(per, 16)), w.n, w.k, e.kind == kEpiPlanes ? max_splits : 1, &bn, &splits);
+    r = launch_tc_any(s, bn, w, am, g.rows, splits, &g, e);
+  }
+  return r == cudaSuccess ? splits : -1;
+}
+
+cudaError_t launch_pack_heads_transposed(cudaStream_t s, const __nv_bfloat16* src, int heads, int dim, int rank, __nv_bfloat16* dst,
+                                         int rankp, int dimp) {
+  lm_pack_heads_transposed_kernel<<<std::min(heads * rank, 148 * 16), 256, 0, s>>>(src, heads, dim, rank, dst, rankp, dimp);
+  return cudaGetLastError();
+}
 cudaError_t launch_pack_rows(cudaStream_t s, const __nv_bfloat16* src, int n, int k, __nv_bfloat16* dst, int ldk, int row_block,
                              int row_block_pad, int row_mul, int row_off, int col_block, int col_block_pad) {
   lm_pack_rows_kernel<<<std::min(n, 148 * 16), 256, 0, s>>>(src, n, k, dst, ldk, row_block, row_block_pad, row_mul, row_off, col_block,

@@ -1,9 +1,9 @@
-// Row operators of the language-model engine: embedding, sandwich norm with residual and causal input convolution,
-// the bookkeeping of a decode step, and the argmax candidates of greedy sampling.
+// Row operators of the language-model engine: embedding, sandwich norm with residual and causal input convolution, norm
+// behind the residual sum (with the choice of experts), the bookkeeping of a decode step, and the argmax candidates of greedy sampling.
 #include <algorithm>
 
 #include "../device_common.cuh"
-#include "lm_state.h"
+#include "lm_route.cuh"
 
 namespace mllmb200 {
 namespace lm {
@@ -35,6 +35,25 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, const float4& v) {
   *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
 }
 
+// columns [c, c + 4) of a row of the sublayer output
+__device__ __forceinline__ float4 load_delta(const Delta& d, int row, int c) {
+  if (!d.mix_w) {
+    const float* p = d.p + (size_t)row * d.ldx + c;
+    float4 v = *reinterpret_cast<const float4*>(p);
+    for (int i = 1; i < d.planes; ++i) v = fma4(1.0f, *reinterpret_cast<const float4*>(p + i * d.plane), v);
+    return v;
+  }
+  float4 v = make_float4(0, 0, 0, 0);
+  for (int k = 0; k < d.top; ++k) {
+    const int pair = row * d.top + k;
+    const float* p = d.p + (size_t)(d.mix_row ? d.mix_row[pair] : pair) * d.ldx + c;
+    float4 y = *reinterpret_cast<const float4*>(p);
+    for (int i = 1; i < d.planes; ++i) y = fma4(1.0f, *reinterpret_cast<const float4*>(p + i * d.plane), y);
+    v = fma4(d.mix_w[pair], y, v);
+  }
+  return v;
+}
+
 // x' = x + rms_unit(delta) * g_post;  h = rms_unit(x') * g_pre;  out = h + conv(h).
 // The gains are one number per norm.  A CTA walks `rows_per_cta` rows in order and keeps the last taps rows of h in
 // shared memory; the taps - 1 rows in front of its first one are recomputed (x_in is not overwritten: x_out is another
@@ -48,7 +67,7 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
   pdl_launch_dependents();
   pdl_wait_prior();
   const int tid = threadIdx.x, nv = a.ldx >> 2;
-  const float g_pre = *a.g_pre, g_post = a.delta ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
+  const float g_pre = *a.g_pre, g_post = a.delta.p ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
   const int r_begin = blockIdx.x * a.rows_per_cta, r_end = min(r_begin + a.rows_per_cta, a.rows);
   int t0 = r_begin;
   if (a.taps > 1) t0 = max(r_begin - (a.taps - 1), a.entries[a.row_entry[r_begin]].row0);
@@ -61,7 +80,7 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
       const int c = tid + i * kNormThreads;
       x[i] = c < nv ? reinterpret_cast<const float4*>(xr)[c] : make_float4(0, 0, 0, 0);
     }
-    if (a.delta) {
+    if (a.delta.p) {
       float4 d[NV];
       float ss = 0.0f;
 #pragma unroll
@@ -69,9 +88,7 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
         const int c = tid + i * kNormThreads;
         d[i] = make_float4(0, 0, 0, 0);
         if (c < nv) {
-          const float* dr = a.delta + (size_t)src * a.ldx + c * 4;
-          d[i] = *reinterpret_cast<const float4*>(dr);
-          for (int p = 1; p < a.planes; ++p) d[i] = fma4(1.0f, *reinterpret_cast<const float4*>(dr + p * a.plane), d[i]);
+          d[i] = load_delta(a.delta, src, c * 4);
           ss += dot4(d[i]);
         }
       }
@@ -130,6 +147,25 @@ __global__ void __launch_bounds__(kNormThreads) lm_norm_kernel(NormArgs a) {
   }
 }
 
+// A row of the sublayer output, column lane + 32 i of float4s in x[i].
+template <int NVW>
+__device__ __forceinline__ void warp_delta(const Delta& d, int row, int lane, int nv, float4 (&x)[NVW]) {
+  const int n_src = d.mix_w ? d.top : 1;
+#pragma unroll
+  for (int i = 0; i < NVW; ++i) x[i] = make_float4(0, 0, 0, 0);
+  for (int k = 0; k < n_src; ++k) {
+    const int pair = row * n_src + k;
+    const float g = d.mix_w ? d.mix_w[pair] : 1.0f;
+    const float* src = d.p + (size_t)(d.mix_w && d.mix_row ? d.mix_row[pair] : pair) * d.ldx;
+    for (int p = 0; p < d.planes; ++p)
+#pragma unroll
+      for (int i = 0; i < NVW; ++i) {
+        const int c = lane + i * 32;
+        if (c < nv) x[i] = fma4(g, *reinterpret_cast<const float4*>(src + p * d.plane + c * 4), x[i]);
+      }
+  }
+}
+
 // The same for many rows: a warp per row for the sums (no block barrier inside), then - with a convolution - the threads
 // sweep the CTA's rows column by column with the last TW - 1 rows of h in registers.  x' of the CTA's own rows is read
 // back from x_out (or x_in when there is nothing to fold in), that of the rows in front of them from shared memory.
@@ -143,7 +179,7 @@ __global__ void __launch_bounds__(kRowsThreads) lm_norm_rows_kernel(NormArgs a) 
   pdl_launch_dependents();
   pdl_wait_prior();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nv = a.ldx >> 2;
-  const float g_pre = *a.g_pre, g_post = a.delta ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
+  const float g_pre = *a.g_pre, g_post = a.delta.p ? *a.g_post : 0.0f, inv_w = 1.0f / (float)a.width;
   const int r_begin = blockIdx.x * a.rows_per_cta, r_end = min(r_begin + a.rows_per_cta, a.rows);
   int t0 = r_begin;
   if (TW > 1) t0 = max(r_begin - (a.taps - 1), a.entries[a.row_entry[r_begin]].row0);
@@ -157,19 +193,8 @@ __global__ void __launch_bounds__(kRowsThreads) lm_norm_rows_kernel(NormArgs a) 
     const float4* xr = reinterpret_cast<const float4*>(a.x_in + (size_t)t * a.ldx);
     float4 x[NVW];
     float ss = 0.0f;
-    if (a.delta) {
-      const float4* dr = reinterpret_cast<const float4*>(a.delta + (size_t)t * a.ldx);
-#pragma unroll
-      for (int i = 0; i < NVW; ++i) {
-        const int c = lane + i * 32;
-        x[i] = c < nv ? dr[c] : make_float4(0, 0, 0, 0);
-      }
-      for (int p = 1; p < a.planes; ++p)
-#pragma unroll
-        for (int i = 0; i < NVW; ++i) {
-          const int c = lane + i * 32;
-          if (c < nv) x[i] = fma4(1.0f, *reinterpret_cast<const float4*>(a.delta + p * a.plane + (size_t)t * a.ldx + c * 4), x[i]);
-        }
+    if (a.delta.p) {
+      warp_delta<NVW>(a.delta, t, lane, nv, x);
 #pragma unroll
       for (int i = 0; i < NVW; ++i) ss += dot4(x[i]);
       const float r = g_post / sqrtf(warp_sum(ss) * inv_w + a.eps);
@@ -203,7 +228,7 @@ __global__ void __launch_bounds__(kRowsThreads) lm_norm_rows_kernel(NormArgs a) 
   if (TW == 1) return;
   __syncthreads();
   const int keep = a.taps - 1;
-  const float* own_x = a.delta ? a.x_out : a.x_in;
+  const float* own_x = a.delta.p ? a.x_out : a.x_in;
   for (int c = tid * 4; c < a.ldx; c += kRowsThreads * 4) {
     float4 w[TW], hist[TW];  // hist[s]: h of s rows ago
 #pragma unroll
@@ -294,12 +319,142 @@ cudaError_t launch_norm_t(cudaStream_t s, const NormArgs& a) {
   return cudaErrorInvalidValue;
 }
 
-__global__ void lm_embed_kernel(const int* __restrict__ tokens, const __nv_bfloat16* __restrict__ table, int width, int ldx,
-                                float* __restrict__ x) {
+// x' = rms_unit(alpha x + delta) * gain, a CTA per row; with a router the CTA goes on to choose the row's experts.
+template <class T, int NV>
+__global__ void __launch_bounds__(kNormThreads) lm_post_norm_kernel(PostNormArgs a) {
+  extern __shared__ __align__(16) float row_x[];  // [ldx], then [experts]; with a router only
+  __shared__ float scratch[32];
+  const int tid = threadIdx.x, nv = a.ldx >> 2, t = blockIdx.x;
+  pdl_launch_dependents();
+  float4 g[NV];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = tid + i * kNormThreads;
+    g[i] = c < nv ? __ldg(reinterpret_cast<const float4*>(a.gain) + c) : make_float4(0, 0, 0, 0);
+  }
+  pdl_wait_prior();
+  const int src = a.gather ? a.gather[t] : t;
+  float4 x[NV];
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = tid + i * kNormThreads;
+    x[i] = make_float4(0, 0, 0, 0);
+    if (c < nv) {
+      const float4 d = a.delta.p ? load_delta(a.delta, src, c * 4) : x[i];
+      x[i] = fma4(a.alpha, *reinterpret_cast<const float4*>(a.x_in + (size_t)src * a.ldx + c * 4), d);
+    }
+    ss += dot4(x[i]);
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)a.width + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = tid + i * kNormThreads;
+    if (c >= nv) continue;
+    const float4 y = make_float4(x[i].x * r * g[i].x, x[i].y * r * g[i].y, x[i].z * r * g[i].z, x[i].w * r * g[i].w);
+    if (a.x_out) store4(a.x_out + (size_t)t * a.ldx + c * 4, y);
+    store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c * 4, y);
+    if (a.router.w) store4(row_x + c * 4, y);
+  }
+  if (!a.router.w) return;
+  __syncthreads();
+  float* z = row_x + a.ldx;
+  const int warp = tid >> 5, lane = tid & 31;
+  for (int e0 = warp; e0 < a.router.experts; e0 += kNormThreads / 16) {  // two experts at a time
+    const int e1 = e0 + kNormThreads / 32;
+    const bool two = e1 < a.router.experts;
+    const __nv_bfloat16 *w0 = a.router.w + (size_t)e0 * a.router.ldw, *w1 = two ? w0 + (size_t)(kNormThreads / 32) * a.router.ldw : w0;
+    float s0 = 0.0f, s1 = 0.0f;
+#pragma unroll 4
+    for (int c = lane * 8; c < a.ldx; c += 256) {
+      const uint4 p = __ldg(reinterpret_cast<const uint4*>(w0 + c)), q = __ldg(reinterpret_cast<const uint4*>(w1 + c));
+      const float4 u = *reinterpret_cast<const float4*>(row_x + c), v = *reinterpret_cast<const float4*>(row_x + c + 4);
+      s0 += dot8(p, u, v);
+      s1 += dot8(q, u, v);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      s0 += __shfl_xor_sync(0xffffffffu, s0, o);
+      s1 += __shfl_xor_sync(0xffffffffu, s1, o);
+    }
+    if (lane == 0) {
+      z[e0] = s0 + a.router.b[e0];
+      if (two) z[e1] = s1 + a.router.b[e1];
+    }
+  }
+  __syncthreads();
+  if (warp == 0) choose_experts(z, a.router, t, lane);
+}
+
+// The same for many rows, a warp per row.
+template <class T, int NVW>
+__global__ void __launch_bounds__(kNormThreads) lm_post_norm_rows_kernel(PostNormArgs a) {
   pdl_launch_dependents();
   pdl_wait_prior();
+  const int lane = threadIdx.x & 31, nv = a.ldx >> 2, t = blockIdx.x * (kNormThreads / 32) + (threadIdx.x >> 5);
+  if (t >= a.rows) return;
+  float4 x[NVW];
+  if (a.delta.p) {
+    warp_delta<NVW>(a.delta, t, lane, nv, x);
+  } else {
+#pragma unroll
+    for (int i = 0; i < NVW; ++i) x[i] = make_float4(0, 0, 0, 0);
+  }
+  const float4* xr = reinterpret_cast<const float4*>(a.x_in + (size_t)t * a.ldx);
+  float ss = 0.0f;
+#pragma unroll
+  for (int i = 0; i < NVW; ++i) {
+    const int c = lane + i * 32;
+    if (c < nv) x[i] = fma4(a.alpha, xr[c], x[i]);
+    ss += dot4(x[i]);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float r = 1.0f / sqrtf(ss / (float)a.width + a.eps);
+#pragma unroll
+  for (int i = 0; i < NVW; ++i) {
+    const int c = lane + i * 32;
+    if (c >= nv) continue;
+    const float4 g = __ldg(reinterpret_cast<const float4*>(a.gain) + c);
+    const float4 y = make_float4(x[i].x * r * g.x, x[i].y * r * g.y, x[i].z * r * g.z, x[i].w * r * g.w);
+    if (a.x_out) store4(a.x_out + (size_t)t * a.ldx + c * 4, y);
+    store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c * 4, y);
+  }
+}
+
+constexpr int kFusedRouterRows = 2 * kSms;
+
+template <class T, int NV>
+cudaError_t launch_post_norm_nv(cudaStream_t s, const PostNormArgs& a) {
+  const size_t smem = a.router.w ? (size_t)(a.ldx + a.router.experts) * sizeof(float) : 0;
+  return launch_pdl(lm_post_norm_kernel<T, NV>, dim3(a.rows), dim3(kNormThreads), smem, s, a);
+}
+template <class T>
+cudaError_t launch_post_norm_t(cudaStream_t s, const PostNormArgs& a) {
+  if (a.rows > kFusedRouterRows && !a.gather && !a.router.w && a.ldx <= 4096) {
+    const int w = (a.ldx / 4 + 31) / 32;
+    const dim3 grid((a.rows + kNormThreads / 32 - 1) / (kNormThreads / 32));
+    if (w <= 8) return launch_pdl(lm_post_norm_rows_kernel<T, 8>, grid, dim3(kNormThreads), 0, s, a);
+    if (w <= 16) return launch_pdl(lm_post_norm_rows_kernel<T, 16>, grid, dim3(kNormThreads), 0, s, a);
+    return launch_pdl(lm_post_norm_rows_kernel<T, 32>, grid, dim3(kNormThreads), 0, s, a);
+  }
+  const int per = (a.ldx / 4 + kNormThreads - 1) / kNormThreads;
+  if (per <= 1) return launch_post_norm_nv<T, 1>(s, a);
+  if (per <= 2) return launch_post_norm_nv<T, 2>(s, a);
+  if (per <= 4) return launch_post_norm_nv<T, 4>(s, a);
+  if (per <= 8) return launch_post_norm_nv<T, 8>(s, a);
+  return cudaErrorInvalidValue;
+}
+
+template <class T>
+__global__ void lm_embed_kernel(const int* __restrict__ tokens, const __nv_bfloat16* __restrict__ table, int width, int ldx,
+                                float* __restrict__ x, T* __restrict__ h, int* __restrict__ zero, int n_zero) {
+  pdl_launch_dependents();
+  pdl_wait_prior();
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n_zero; i += gridDim.x * blockDim.x) zero[i] = 0;
   const __nv_bfloat16* src = table + (size_t)tokens[blockIdx.x] * width;
   float* dst = x + (size_t)blockIdx.x * ldx;
+  T* hd = h ? h + (size_t)blockIdx.x * ldx : nullptr;
   int k0 = 0;
   if ((width & 7) == 0) {
     k0 = width;
@@ -307,12 +462,19 @@ __global__ void lm_embed_kernel(const int* __restrict__ tokens, const __nv_bfloa
       const uint4 p = *reinterpret_cast<const uint4*>(src + k);
       const uint32_t w[4] = {p.x, p.y, p.z, p.w};
 #pragma unroll
-      for (int i = 0; i < 2; ++i)
-        store4(dst + k + 4 * i, make_float4(__uint_as_float(w[2 * i] << 16), __uint_as_float(w[2 * i] & 0xffff0000u),
-                                            __uint_as_float(w[2 * i + 1] << 16), __uint_as_float(w[2 * i + 1] & 0xffff0000u)));
+      for (int i = 0; i < 2; ++i) {
+        const float4 v = make_float4(__uint_as_float(w[2 * i] << 16), __uint_as_float(w[2 * i] & 0xffff0000u),
+                                     __uint_as_float(w[2 * i + 1] << 16), __uint_as_float(w[2 * i + 1] & 0xffff0000u));
+        store4(dst + k + 4 * i, v);
+        if (hd) store4(hd + k + 4 * i, v);
+      }
     }
   }
-  for (int k = k0 + threadIdx.x; k < ldx; k += blockDim.x) dst[k] = k < width ? __bfloat162float(src[k]) : 0.0f;
+  for (int k = k0 + threadIdx.x; k < ldx; k += blockDim.x) {
+    const float v = k < width ? __bfloat162float(src[k]) : 0.0f;
+    dst[k] = v;
+    if (hd) hd[k] = static_cast<T>(v);  // exact: the table is bf16
+  }
 }
 
 // Rows of a decode step: one token per slot, from the slots' own state.
@@ -363,8 +525,15 @@ __global__ void __launch_bounds__(256) lm_argmax_kernel(const float* __restrict_
 cudaError_t launch_norm(cudaStream_t s, bool f32, const NormArgs& a) {
   return f32 ? launch_norm_t<float>(s, a) : launch_norm_t<__nv_bfloat16>(s, a);
 }
-cudaError_t launch_embed(cudaStream_t s, const int* tokens, const __nv_bfloat16* table, int width, int ldx, int rows, float* x) {
-  return launch_pdl(lm_embed_kernel, dim3(rows), dim3(256), 0, s, tokens, table, width, ldx, x);
+bool fused_router(int rows) { return rows <= kFusedRouterRows; }
+cudaError_t launch_post_norm(cudaStream_t s, bool f32, const PostNormArgs& a) {
+  return f32 ? launch_post_norm_t<float>(s, a) : launch_post_norm_t<__nv_bfloat16>(s, a);
+}
+cudaError_t launch_embed(cudaStream_t s, bool f32, const int* tokens, const __nv_bfloat16* table, int width, int ldx, int rows, float* x,
+                         void* h, int* zero, int n_zero) {
+  if (f32) return launch_pdl(lm_embed_kernel<float>, dim3(rows), dim3(256), 0, s, tokens, table, width, ldx, x, static_cast<float*>(h), zero, n_zero);
+  return launch_pdl(lm_embed_kernel<__nv_bfloat16>, dim3(rows), dim3(256), 0, s, tokens, table, width, ldx, x, static_cast<__nv_bfloat16*>(h), zero,
+                    n_zero);
 }
 cudaError_t launch_decode_prep(cudaStream_t s, int n, const int* slots, const int* pos, const int* token, const int* flip,
                                int2* row_sp, int* row_token, Entry* entries, int* row_entry) {

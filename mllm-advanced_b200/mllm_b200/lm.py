@@ -9,22 +9,25 @@ import numpy as np
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 BF16, F32 = 0, 1
-ATTENTION, RETENTION = 0, 1
+ATTENTION, RETENTION, LATENT = 0, 1, 2
+CLAMPED, GELU, SILU = 0, 1, 2  # gated feed-forwards
+NORM_SANDWICH, NORM_POST = 0, 1
 TENSORS = {n: i for i, n in enumerate(("q", "k", "v", "g", "o", "gate", "up", "down", "norm1", "norm1b", "norm2", "norm2b",
-                                       "conv", "rel", "decay"))}
+                                       "conv", "rel", "decay", "dkv", "dkv_norm", "uk", "uv", "router", "router_b"))}
 MODEL_TENSORS = {"embed": 100, "head": 101, "final_norm": 102}
-_LINEARS = {"q", "k", "v", "g", "o", "gate", "up", "down", "embed", "head"}
+_LINEARS = {"q", "k", "v", "g", "o", "gate", "up", "down", "embed", "head", "dkv", "uk", "uv", "router"}
 
 
 class Config(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("vocab", "width", "layers", "dtype", "conv_taps", "max_seqs", "max_ctx", "max_rows")] + \
-               [("eps", C.c_float), ("logit_scale", C.c_float)]
+               [("eps", C.c_float), ("logit_scale", C.c_float), ("norm_place", C.c_int), ("residual_scale", C.c_float)]
 
 
 class Layer(C.Structure):
     _fields_ = [(n, C.c_int) for n in ("mixer", "heads", "kv_heads", "dim", "vdim")] + [("score_scale", C.c_float)] + \
                [(n, C.c_int) for n in ("sink", "bias_rows", "bias_max", "rot_dims")] + [("rot_base", C.c_double), ("ff", C.c_int),
-                                                                                      ("ff_limit", C.c_float), ("weights_of", C.c_int)]
+                                                                                      ("ff_limit", C.c_float), ("weights_of", C.c_int)] + \
+               [(n, C.c_int) for n in ("kv_rank", "kv_from", "act", "experts", "top")]
 
 
 class EngineError(RuntimeError):
@@ -54,6 +57,7 @@ def lib():
     L = C.CDLL(lib_path())
     vp, ci = C.c_void_p, C.c_int
     sig = {"create": [C.POINTER(Config), C.POINTER(Layer), C.POINTER(vp)], "set_tensor": [vp, ci, ci, vp, ci, ci],
+           "set_expert": [vp, ci, ci, ci, vp, ci, ci],
            "step": [vp, ci, vp, vp, vp, ci, vp, vp, ci], "decode": [vp, ci, vp, ci], "free_slot": [vp, ci],
            "read": [vp, ci, ci, ci, vp, vp], "keep_residual": [vp, ci], "read_residual": [vp, ci, ci, vp],
            "stats": [vp, C.POINTER(C.c_size_t), C.POINTER(C.c_longlong)], "synchronize": [vp], "check_device_status": [vp],
@@ -85,9 +89,9 @@ class LanguageModel:
     """config: fields of Config without `layers` and `dtype`; layers: one dict of Layer fields per layer."""
 
     def __init__(self, config, layers, dtype=BF16):
-        self.config = dict(config, layers=len(layers), dtype=dtype)
+        self.config = dict({"norm_place": NORM_SANDWICH, "residual_scale": 1.0}, **config, layers=len(layers), dtype=dtype)
         self.layers = [dict({"sink": 0, "bias_rows": 0, "bias_max": 0, "rot_dims": 0, "rot_base": 1.0, "ff": 0, "ff_limit": 0.0,
-                             "score_scale": 1.0, "weights_of": -1}, **d) for d in layers]
+                             "score_scale": 1.0, "weights_of": -1, "kv_rank": 0, "kv_from": -1, "act": CLAMPED, "experts": 0, "top": 0}, **d) for d in layers]
         self.vocab, self.max_seqs = self.config["vocab"], self.config["max_seqs"]
         self.max_ctx, self.max_rows = self.config["max_ctx"], self.config["max_rows"]
         self._L, self._h = lib(), C.c_void_p()
@@ -114,10 +118,9 @@ class LanguageModel:
             raise EngineError(st, where, self._L.mllmb200_lm_last_error(self._h).decode())
 
     # ---- weights
-    def set_tensor(self, layer, name, data):
-        """layer -1: a tensor of the model.  numpy (bf16 as uint16 bits for the linear maps), or a torch tensor on the
-        device (bf16 for the linear maps)."""
-        which = (MODEL_TENSORS if layer < 0 else TENSORS)[name]
+    @staticmethod
+    def _tensor(name, data):
+        """(what keeps the memory, address, rows, columns)"""
         if isinstance(data, (np.ndarray, np.generic)):
             data = np.ascontiguousarray(data, np.uint16 if name in _LINEARS else np.float64 if name == "decay" else np.float32)
             ptr, shape = data.ctypes.data, data.shape
@@ -125,7 +128,20 @@ class LanguageModel:
             data = data.contiguous()
             ptr, shape = data.data_ptr(), tuple(data.shape)
         rows, cols = shape if len(shape) == 2 else (1, int(np.prod(shape)))
+        return data, ptr, rows, cols
+
+    def set_tensor(self, layer, name, data):
+        """layer -1: a tensor of the model.  numpy (bf16 as uint16 bits for the linear maps), or a torch tensor on the
+        device (bf16 for the linear maps)."""
+        which = (MODEL_TENSORS if layer < 0 else TENSORS)[name]
+        data, ptr, rows, cols = self._tensor(name, data)
         self._check(self._L.mllmb200_lm_set_tensor(self._h, layer, which, ptr, rows, cols), f"tensor {name} of layer {layer}")
+
+    def set_expert(self, layer, expert, name, data):
+        """gate, up or down of one expert of a mixture."""
+        data, ptr, rows, cols = self._tensor(name, data)
+        self._check(self._L.mllmb200_lm_set_expert(self._h, layer, expert, TENSORS[name], ptr, rows, cols),
+                    f"tensor {name} of expert {expert} of layer {layer}")
 
     # ---- slots
     def acquire(self):

@@ -8,7 +8,7 @@ import os
 
 import numpy as np
 
-from . import lm, vupuzen
+from . import lm, taralix, vupuzen
 from .safetensors import Tensors
 
 DTYPES = {"bfloat16": lm.BF16, "float32": lm.F32}
@@ -16,6 +16,10 @@ DTYPES = {"bfloat16": lm.BF16, "float32": lm.F32}
 
 def _load_vupuzen(cfg, folder, dtype, max_seqs, max_ctx, max_rows):
     return vupuzen.load(cfg, Tensors(folder), DTYPES[dtype], max_seqs, max_ctx, max_rows)
+
+
+def _load_taralix(cfg, folder, dtype, max_seqs, max_ctx, max_rows):
+    return taralix.load(cfg, Tensors(folder), DTYPES[dtype], max_seqs, max_ctx, max_rows)
 
 
 def _load_qwen2(cfg, folder, dtype, max_seqs, max_ctx, max_rows):
@@ -46,6 +50,7 @@ def _load_qwen2(cfg, folder, dtype, max_seqs, max_ctx, max_rows):
 
 MODELS = {  # design -> (runtime, number formats, loader)
     vupuzen.ARCHITECTURE: ("engine", ("bfloat16", "float32"), _load_vupuzen),
+    taralix.ARCHITECTURE: ("engine", ("bfloat16", "float32"), _load_taralix),
     "Qwen2ForCausalLM": ("qwen2", ("w4a32",), _load_qwen2),
 }
 
