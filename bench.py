@@ -1366,10 +1366,11 @@ def main():
                     help="with --prefill-only: (q,k,v) and (gate,up) as grouped calls, fastest policy")
     ap.add_argument("--prefill-f16", action="store_true", help="with --prefill-only: use the fp16 tensor-core path (kernel 4)")
     ap.add_argument("--fast-prefill", action="store_true", help="time the prefill linears on 2 layers instead of 28")
-    ap.add_argument("--lm", action="store_true", help="only the language-model engine: Vupuzen beside the Qwen2 decoder at equal layer sizes")
-    ap.add_argument("--lm-size", default=None, help="with --lm: one of 0.5b, 1.5b, 2048")
-    ap.add_argument("--lm-no-compare", action="store_true", help="with --lm: without the Qwen2 decoder")
-    ap.add_argument("--lm-once", default=None, choices=["vupuzen", "qwen2"], help="with --lm: a short untimed run (for launch lists)")
+    ap.add_argument("--lm", action="store_true", help="only the language-model engine: a design beside the closest other model at equal layer sizes")
+    ap.add_argument("--lm-design", default="vupuzen", choices=["vupuzen", "taralix"], help="with --lm: Vupuzen beside the Qwen2 decoder, or Taralix beside Vupuzen")
+    ap.add_argument("--lm-size", default=None, help="with --lm: one of 0.5b, 1.5b, 2048 (Vupuzen) or 0.5b, 1.5b, moe (Taralix)")
+    ap.add_argument("--lm-no-compare", action="store_true", help="with --lm: without the other model")
+    ap.add_argument("--lm-once", default=None, choices=["vupuzen", "taralix", "qwen2"], help="with --lm: a short untimed run (for launch lists)")
     args = ap.parse_args()
     # Libraries write to file descriptor 1 behind Python's back (NCCL prints its version banner there when a
     # communicator is created); stdout must carry the result lines only, so everything that is not printed

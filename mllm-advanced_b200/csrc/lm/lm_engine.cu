@@ -67,6 +67,7 @@ struct StepCtx {
 struct Engine {
   mllmb200_lm_config c{};
   bool f32 = false, post = false, latent = false;
+  bool absorb_all = false;  // all rows attend through the latent: 32-bit mode, heads too large for the prompt kernel
   int elt = 2, widthp = 0, plane_rows = 0, logit_rows = 0, max_splits_ctx = 1;
   std::vector<LayerState> layers;
   __nv_bfloat16* embed = nullptr;
@@ -194,7 +195,8 @@ int check_layer(Engine* e, int i, const mllmb200_lm_layer& d) {
     return fail(e, MLLMB200_UNSUPPORTED, "layer %d: mixer %d", i, d.mixer);
   if (d.heads < 1 || d.kv_heads < 1 || d.heads % d.kv_heads || d.dim < 1 || d.vdim < 1 || d.ff < 0)
     return fail(e, MLLMB200_INVALID_ARG, "layer %d: sizes", i);
-  if (d.dim > 256 || d.vdim > 256 || d.heads / d.kv_heads > 64) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: head sizes beyond 256 or more than 64 heads per key", i);
+  const int most = d.mixer == MLLMB200_LM_LATENT ? kMaxRank : 256;
+  if (d.dim > most || d.vdim > most || d.heads / d.kv_heads > 64) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: head sizes beyond %d or more than 64 heads per key", i, most);
   if (d.act < MLLMB200_LM_ACT_CLAMPED || d.act > MLLMB200_LM_ACT_SILU) return fail(e, MLLMB200_UNSUPPORTED, "layer %d: activation %d", i, d.act);
   if (d.experts) {
     if (d.experts < 1 || d.top < 1 || d.top > d.experts || d.ff < 1) return fail(e, MLLMB200_INVALID_ARG, "layer %d: %d of %d experts", i, d.top, d.experts);
@@ -290,6 +292,7 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
       heads = std::max(heads, (size_t)L.d.heads);
     } else if (is_latent(L)) {
       e->latent = true;
+      e->absorb_all = e->absorb_all || e->f32 || L.d.dim > 256 || L.d.vdim > 256;
       if (owns_latent(L)) {
         LM_OK(dalloc_bytes(e, &L.kc, slots * c.max_ctx * L.rankp * e->elt, true));
         if (make_act_map(&L.a_kc, L.kc, (int)(slots * c.max_ctx), L.rankp) != MLLMB200_OK) return fail(e, MLLMB200_CUDA_ERROR, "tensor map of a latent cache");
@@ -327,7 +330,7 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
   }
   e->plane_rows = std::max(e->plane_rows, (int)(rows * top));
   if (e->latent) {
-    e->latent_cap = e->f32 ? c.max_rows : std::min(c.max_rows, c.max_seqs * kAbsorbMax);
+    e->latent_cap = e->absorb_all ? c.max_rows : std::min(c.max_rows, c.max_seqs * kAbsorbMax);
     LM_OK(dalloc(e, &e->fresh, rows * rank));
     LM_OK(dalloc_bytes(e, &e->qa, e->latent_cap * head_rank * e->elt));
     if (e->f32) {
@@ -335,9 +338,11 @@ int create(Engine* e, const mllmb200_lm_layer* descs) {
     } else {
       LM_OK(dalloc(e, &e->lat_part, latent_parts(e->latent_cap) * head_rank));
       LM_OK(dalloc(e, &e->lat_ml, latent_parts(e->latent_cap) * lat_heads));
-      e->expand_cap = c.max_ctx + (c.max_seqs > 1 ? c.max_rows : 0);
-      LM_OK(dalloc_bytes(e, &e->ex_k, e->expand_cap * ex_k * e->elt));
-      LM_OK(dalloc_bytes(e, &e->ex_v, e->expand_cap * ex_v * e->elt));
+      if (!e->absorb_all) {
+        e->expand_cap = c.max_ctx + (c.max_seqs > 1 ? c.max_rows : 0);
+        LM_OK(dalloc_bytes(e, &e->ex_k, e->expand_cap * ex_k * e->elt));
+        LM_OK(dalloc_bytes(e, &e->ex_v, e->expand_cap * ex_v * e->elt));
+      }
     }
   }
   if (experts) {
@@ -1128,7 +1133,7 @@ int step(Engine* e, int n_entries, const int* slots, const int* counts, const in
   if (e->latent)
     for (const Entry& en : entries) {
       const int ctx = en.pos0 + en.count;
-      if (e->f32 || en.count <= kAbsorbMax) {
+      if (e->absorb_all || en.count <= kAbsorbMax) {
         for (int j = 0; j < en.count; ++j) latent_rows.push_back(en.row0 + j);
         latent_ctx = std::max(latent_ctx, ctx);
         continue;

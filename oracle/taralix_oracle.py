@@ -103,6 +103,20 @@ def forward(cfg, weights, tokens, want_layers=False):
     return (logits, np.stack(layers)) if want_layers else logits
 
 
+def router_gaps(cfg, weights, tokens):
+    """Per token, the smallest distance over all layers between the last chosen and the first rejected router logit."""
+    w = {k: np.asarray(v, np.float64) for k, v in weights.items()}
+    x, latents, gap = w["embed"][np.asarray(tokens)], {}, np.full(len(tokens), np.inf)
+    for i, e in enumerate(cfg["layers"]):
+        if e.get("mlp") and e["mlp"]["kind"] == "moe" and e["mlp"]["router"]["top"] < e["mlp"]["router"]["experts"]:
+            mid = layer_forward(x, i, w, dict(cfg, layers=[dict(a, mlp=None) for a in cfg["layers"]]), dict(latents))
+            z = np.sort(mid @ w[f"l{i}.mlp.router"].T + w[f"l{i}.mlp.router.b"], axis=-1)[:, ::-1]
+            top = e["mlp"]["router"]["top"]
+            gap = np.minimum(gap, z[:, top - 1] - z[:, top])
+        x = layer_forward(x, i, w, cfg, latents)
+    return gap
+
+
 def greedy(cfg, weights, tokens, steps):
     """Tokens of greedy decoding, recomputing the whole sequence every step (lowest index on ties)."""
     seq = list(tokens)

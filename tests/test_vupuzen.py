@@ -10,56 +10,18 @@ import pytest
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 sys.path.insert(0, os.path.join(ROOT, "oracle"))
 
+import lm_case  # noqa: E402
 import lm_models as M  # noqa: E402
 import vupuzen_oracle as V  # noqa: E402
+from lm_case import BAR, DTYPES, residual_after, row_error  # noqa: E402
 from mllm_b200 import lm, registry, replay, scheduler  # noqa: E402
 
 gpu = pytest.mark.gpu
-# relative rms error of a row of logits; bf16: a few roundings of 2^-9 per layer.  A retention head divided by a root mean
-# square that happens to be small (its first terms nearly cancel) enlarges them: one row in fifty may reach OUTLIER.
-BAR = {"float32": 3e-5, "bfloat16": 0.06}
-OUTLIER = {"float32": 1e-4, "bfloat16": 0.2}
-DTYPES = ["float32", "bfloat16"]
 
 
-def row_error(got, want):
-    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
-    return np.sqrt(np.mean((got - want) ** 2, axis=-1)) / np.sqrt(np.mean(want ** 2))
-
-
-class Case:
-    """A model on the GPU and in the oracle."""
-
-    def __init__(self, folder, cfg, w, dtype, max_seqs=6, max_ctx=1024, max_rows=1024):
-        self.cfg, self.w, self.dtype = cfg, w, dtype
-        self.model, runtime = registry.load(M.write(folder, cfg, w), dtype, max_seqs, max_ctx, max_rows)
-        assert runtime == "engine"
-
-    def oracle(self, tokens):
-        return V.forward(self.cfg, self.w, tokens)
-
-    def tokens(self, n, seed=0):
-        return np.random.default_rng(seed + 1000).integers(0, self.cfg["vocab"], n).tolist()
-
-    def run(self, tokens, portions=None, slot=None):
-        """Logits of every place, read in the given portions (the last one is repeated)."""
-        own = slot is None
-        slot = self.model.acquire() if own else slot
-        out, at, k = [], 0, 0
-        portions = portions or [len(tokens)]
-        while at < len(tokens):
-            n = min(portions[min(k, len(portions) - 1)], len(tokens) - at)
-            out.append(self.model.step([(slot, tokens[at:at + n])], list(range(n))))
-            at, k = at + n, k + 1
-        if own:
-            self.model.release(slot)
-        self.model.check_device_status()
-        return np.concatenate(out)
-
-    def check(self, got, want):
-        e = row_error(got, want)
-        over = int((e >= BAR[self.dtype]).sum())
-        assert over <= len(e) // 50 and e.max() < OUTLIER[self.dtype], (float(e.max()), int(e.argmax()), over, len(e))
+class Case(lm_case.Case):
+    def __init__(self, folder, cfg, w, dtype, *sizes, **kw):
+        super().__init__(M.write(folder, cfg, w), V, cfg, w, dtype, *sizes, **kw)
 
 
 @pytest.fixture(scope="module")
@@ -210,21 +172,6 @@ def one_layer(kind, mixer, ff=None, taps=1, width=96, vocab=64, seed=1, conv=0.0
     w = M.weights(cfg, seed, rel_rows=rel_rows)
     w["l0.canon1"] = M.rounded(np.random.default_rng(seed).standard_normal((width, taps)) * conv)
     return cfg, w
-
-
-def residual_after(case, tokens, portions=None):
-    """Residual stream after layer 0, per token."""
-    m, out, at = case.model, [], 0
-    slot = m.acquire()
-    m.keep_residual(True)
-    for n in portions or [len(tokens)]:
-        m.step([(slot, tokens[at:at + n])])
-        out.append(m.residual(0, n))
-        at += n
-    m.keep_residual(False)
-    m.release(slot)
-    assert at == len(tokens)
-    return np.concatenate(out)
 
 
 MECHANISMS = {
