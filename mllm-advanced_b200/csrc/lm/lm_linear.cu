@@ -29,12 +29,17 @@ __device__ __forceinline__ float from_f32<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
+// All forms are g sigmoid(z(g)) times a form of u: 0.5 (1 + tanh(x)) = sigmoid(2 x).
 __device__ __forceinline__ float gated(const Epi& e, float g, float u) {
-  if (e.act_kind == MLLMB200_LM_ACT_GELU) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
-  if (e.act_kind == MLLMB200_LM_ACT_SILU) return g / (1.0f + expf(-g)) * u;
-  g = fminf(g, e.limit);
-  u = fminf(fmaxf(u, -e.limit), e.limit);
-  return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+  float z = g;
+  if (e.act_kind == MLLMB200_LM_ACT_GELU) {
+    z = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+  } else if (e.act_kind == MLLMB200_LM_ACT_CLAMPED) {
+    g = fminf(g, e.limit);
+    u = fminf(fmaxf(u, -e.limit), e.limit) + 1.0f;
+    z = 1.702f * g;
+  }
+  return g / (1.0f + expf(-z)) * u;
 }
 
 // address of column n of row m of a q|k|v product
@@ -433,7 +438,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
       const int m = m0 + quarter * 32 + lane;
       if (m0 + quarter * 32 < m_end) {
         const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16) + buf * BN;
-#pragma unroll
+#pragma unroll 1  // the epilogue's code is long enough
         for (int c = 0; c < BN; c += 32) {
           if (n0 + c >= N) break;
           uint32_t r0[16], r1[16];
