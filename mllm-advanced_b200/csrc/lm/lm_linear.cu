@@ -30,16 +30,22 @@ template <>
 __device__ __forceinline__ __nv_bfloat16 from_f32<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 
 // All forms are g sigmoid(z(g)) times a form of u: 0.5 (1 + tanh(x)) = sigmoid(2 x).
-__device__ __forceinline__ float gated(const Epi& e, float g, float u) {
+template <int ACT>
+__device__ __forceinline__ float gated_as(float limit, float g, float u) {
   float z = g;
-  if (e.act_kind == MLLMB200_LM_ACT_GELU) {
+  if (ACT == MLLMB200_LM_ACT_GELU) {
     z = 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
-  } else if (e.act_kind == MLLMB200_LM_ACT_CLAMPED) {
-    g = fminf(g, e.limit);
-    u = fminf(fmaxf(u, -e.limit), e.limit) + 1.0f;
+  } else if (ACT == MLLMB200_LM_ACT_CLAMPED) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.0f;
     z = 1.702f * g;
   }
   return g / (1.0f + expf(-z)) * u;
+}
+__device__ __forceinline__ float gated(const Epi& e, float g, float u) {
+  return e.act_kind == MLLMB200_LM_ACT_GELU   ? gated_as<MLLMB200_LM_ACT_GELU>(e.limit, g, u)
+         : e.act_kind == MLLMB200_LM_ACT_SILU ? gated_as<MLLMB200_LM_ACT_SILU>(e.limit, g, u)
+                                              : gated_as<MLLMB200_LM_ACT_CLAMPED>(e.limit, g, u);
 }
 
 // address of column n of row m of a q|k|v product
@@ -79,9 +85,21 @@ __device__ __forceinline__ uint32_t pack_bf16(float a, float b) {
   return *reinterpret_cast<const uint32_t*>(&h);
 }
 
-// columns [n, n + 16) of row m (n a multiple of 16), bf16 outputs
+// eight gated pairs, the first of them columns (n, n + 1); pairs past N write zeros into the padding of the row
+template <int ACT>
+__device__ __forceinline__ void gate8(const Epi& e, int m, int n, int N, const float (&v)[16]) {
+  float a[8];
+#pragma unroll
+  for (int i = 0; i < 8; ++i) a[i] = n + 2 * i < N ? gated_as<ACT>(e.limit, v[2 * i], v[2 * i + 1]) : 0.0f;
+  *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(e.act) + (size_t)m * e.ld_act + (n >> 1)) =
+      make_uint4(pack_bf16(a[0], a[1]), pack_bf16(a[2], a[3]), pack_bf16(a[4], a[5]), pack_bf16(a[6], a[7]));
+}
+
+// columns [n, n + 16) of row m (n a multiple of 16), bf16 outputs; FORM: see form_of
+enum Form { kFormPlanes, kFormScatter, kFormGate };
+template <int FORM>
 __device__ __forceinline__ void store16(const Epi& e, int m, int n, int N, const float (&v)[16], int split) {
-  if (e.kind == kEpiPlanes) {
+  if (FORM == kFormPlanes) {
     float* y = e.y + (size_t)split * e.plane + (size_t)m * e.ldy + n;
     if (n + 16 <= N && (e.ldy & 3) == 0) {
 #pragma unroll
@@ -93,22 +111,25 @@ __device__ __forceinline__ void store16(const Epi& e, int m, int n, int N, const
       for (int i = 0; i < 16; ++i)
         if (n + i < N) y[i] = v[i] * e.scale;
     }
-  } else if (e.kind == kEpiQLatent && n >= e.q_end) {
-    float4* y = reinterpret_cast<float4*>(e.y + (size_t)m * e.ldy + (n - e.q_end));
+  } else if (FORM == kFormScatter) {
+    if (e.kind == kEpiQLatent && n >= e.q_end) {
+      float4* y = reinterpret_cast<float4*>(e.y + (size_t)m * e.ldy + (n - e.q_end));
 #pragma unroll
-    for (int i = 0; i < 4; ++i) y[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
-  } else if (e.kind != kEpiGate) {  // head sizes are multiples of 16: the chunk lies in one head
-    uint4* p = reinterpret_cast<uint4*>(qkv_ptr<__nv_bfloat16>(e, m, n));
-    p[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
-    p[1] = make_uint4(pack_bf16(v[8], v[9]), pack_bf16(v[10], v[11]), pack_bf16(v[12], v[13]), pack_bf16(v[14], v[15]));
-  } else {  // pairs past N write zeros into the padding of the row
-    float a[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) a[i] = n + 2 * i < N ? gated(e, v[2 * i], v[2 * i + 1]) : 0.0f;
-    *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(e.act) + (size_t)m * e.ld_act + (n >> 1)) =
-        make_uint4(pack_bf16(a[0], a[1]), pack_bf16(a[2], a[3]), pack_bf16(a[4], a[5]), pack_bf16(a[6], a[7]));
+      for (int i = 0; i < 4; ++i) y[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+    } else {  // head sizes are multiples of 16: the chunk lies in one head
+      uint4* p = reinterpret_cast<uint4*>(qkv_ptr<__nv_bfloat16>(e, m, n));
+      p[0] = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+      p[1] = make_uint4(pack_bf16(v[8], v[9]), pack_bf16(v[10], v[11]), pack_bf16(v[12], v[13]), pack_bf16(v[14], v[15]));
+    }
+  } else if (e.act_kind == MLLMB200_LM_ACT_GELU) {
+    gate8<MLLMB200_LM_ACT_GELU>(e, m, n, N, v);
+  } else if (e.act_kind == MLLMB200_LM_ACT_SILU) {
+    gate8<MLLMB200_LM_ACT_SILU>(e, m, n, N, v);
+  } else {
+    gate8<MLLMB200_LM_ACT_CLAMPED>(e, m, n, N, v);
   }
 }
+Form form_of(const Epi& e) { return e.kind == kEpiPlanes ? kFormPlanes : e.kind == kEpiGate ? kFormGate : kFormScatter; }
 
 // ------------------------------------------------------------------------------------------ GEMV
 constexpr int kGemvThreads = 256, kGemvWarps = kGemvThreads / 32, kGemvUnroll = 4;
@@ -297,7 +318,7 @@ __device__ __forceinline__ uint64_t swizzled_desc(uint32_t addr) {
 // Work items are (K split, weight tile, row tile), row tiles fastest; CTA c takes items c, c + gridDim.x, ...
 // GROUPED: the row tiles are those of `tiles`; whole tiles are copied through amap (boxes of 128 rows), the others through
 // amap16 (16 rows).  Weight tiles and boxes may reach into the next group: those sums are not stored.
-template <int BN, bool GROUPED>
+template <int BN, bool GROUPED, int FORM>
 __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_constant__ CUtensorMap amap,
                                                                    const __grid_constant__ CUtensorMap amap16,
                                                                    const __grid_constant__ CUtensorMap wmap, int a_box, int M, int N,
@@ -438,7 +459,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
       const int m = m0 + quarter * 32 + lane;
       if (m0 + quarter * 32 < m_end) {
         const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16) + buf * BN;
-#pragma unroll 1  // the epilogue's code is long enough
+#pragma unroll 1  // a kernel starts with a cold instruction cache: short code
         for (int c = 0; c < BN; c += 32) {
           if (n0 + c >= N) break;
           uint32_t r0[16], r1[16];
@@ -449,11 +470,11 @@ __global__ void __launch_bounds__(kTcThreads, 1) lm_gemm_tc_kernel(const __grid_
           if (m < m_end) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r0[i]);
-            store16(e, m, n0 + c, N, v, split);
+            store16<FORM>(e, m, n0 + c, N, v, split);
             if (n0 + c + 16 < N) {
 #pragma unroll
               for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r1[i]);
-              store16(e, m, n0 + c + 16, N, v, split);
+              store16<FORM>(e, m, n0 + c + 16, N, v, split);
             }
           }
           __syncwarp();
@@ -526,16 +547,34 @@ void choose_tile(int M, int mt, int a_rows, int N, int K, int max_splits, int* b
   }
 }
 
-template <int BN>
-cudaError_t launch_tc(cudaStream_t s, const Linear& w, const ActMap& am, int M, int splits, const Groups* g, const Epi& e) {
+template <int BN, int FORM>
+cudaError_t launch_tc_form(cudaStream_t s, const Linear& w, const ActMap& am, int M, int splits, const Groups* g, const Epi& e) {
   const int nt = (w.n + BN - 1) / BN;
   const CUtensorMap& wmap = BN < 128 ? w.map32 : w.map128;
   if (g)
-    return launch_pdl(lm_gemm_tc_kernel<BN, true>, dim3(std::min(g->max_tiles * nt * splits, kSms)), dim3(kTcThreads), TcShape<BN>::kSmem, s,
-                      am.map128, am.map16, wmap, 128, M, w.n, w.k, splits, g->tiles, g->n_tiles, g->max_tiles, e);
+    return launch_pdl(lm_gemm_tc_kernel<BN, true, FORM>, dim3(std::min(g->max_tiles * nt * splits, kSms)), dim3(kTcThreads), TcShape<BN>::kSmem,
+                      s, am.map128, am.map16, wmap, 128, M, w.n, w.k, splits, g->tiles, g->n_tiles, g->max_tiles, e);
   const int mt = (M + kTileM - 1) / kTileM;
-  return launch_pdl(lm_gemm_tc_kernel<BN, false>, dim3(std::min(mt * nt * splits, kSms)), dim3(kTcThreads), TcShape<BN>::kSmem, s,
+  return launch_pdl(lm_gemm_tc_kernel<BN, false, FORM>, dim3(std::min(mt * nt * splits, kSms)), dim3(kTcThreads), TcShape<BN>::kSmem, s,
                     M >= kTileM ? am.map128 : am.map16, am.map16, wmap, M >= kTileM ? 128 : 16, M, w.n, w.k, splits, nullptr, nullptr, 0, e);
+}
+template <int BN>
+cudaError_t launch_tc(cudaStream_t s, const Linear& w, const ActMap& am, int M, int splits, const Groups* g, const Epi& e) {
+  const Form f = form_of(e);
+  return f == kFormPlanes ? launch_tc_form<BN, kFormPlanes>(s, w, am, M, splits, g, e)
+         : f == kFormGate ? launch_tc_form<BN, kFormGate>(s, w, am, M, splits, g, e)
+                          : launch_tc_form<BN, kFormScatter>(s, w, am, M, splits, g, e);
+}
+template <int BN, int FORM>
+cudaError_t configure_tc() {
+  const cudaError_t r = cudaFuncSetAttribute(lm_gemm_tc_kernel<BN, false, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcShape<BN>::kSmem);
+  return r != cudaSuccess ? r : cudaFuncSetAttribute(lm_gemm_tc_kernel<BN, true, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, TcShape<BN>::kSmem);
+}
+template <int BN>
+cudaError_t configure_tc_forms() {
+  cudaError_t r = configure_tc<BN, kFormPlanes>();
+  if (r == cudaSuccess) r = configure_tc<BN, kFormScatter>();
+  return r != cudaSuccess ? r : configure_tc<BN, kFormGate>();
 }
 
 template <class T, int MT>
@@ -573,18 +612,10 @@ cudaError_t configure_gemv() {
 }  // namespace
 
 cudaError_t linear_configure() {
-  cudaError_t r = cudaSuccess;
-  auto set = [&](auto f, int bytes) {
-    if (r == cudaSuccess) r = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes);
-  };
-  set(lm_gemm_tc_kernel<256, false>, TcShape<256>::kSmem);
-  set(lm_gemm_tc_kernel<128, false>, TcShape<128>::kSmem);
-  set(lm_gemm_tc_kernel<64, false>, TcShape<64>::kSmem);
-  set(lm_gemm_tc_kernel<32, false>, TcShape<32>::kSmem);
-  set(lm_gemm_tc_kernel<256, true>, TcShape<256>::kSmem);
-  set(lm_gemm_tc_kernel<128, true>, TcShape<128>::kSmem);
-  set(lm_gemm_tc_kernel<64, true>, TcShape<64>::kSmem);
-  set(lm_gemm_tc_kernel<32, true>, TcShape<32>::kSmem);
+  cudaError_t r = configure_tc_forms<256>();
+  if (r == cudaSuccess) r = configure_tc_forms<128>();
+  if (r == cudaSuccess) r = configure_tc_forms<64>();
+  if (r == cudaSuccess) r = configure_tc_forms<32>();
   if (r == cudaSuccess) r = configure_gemv<float>();
   if (r == cudaSuccess) r = configure_gemv<__nv_bfloat16>();
   return r;
