@@ -8,10 +8,12 @@
 //     in fragment order (k is permuted alike on both sides).  It makes the queries U_h^T q_h - some CTAs put the step's
 //     latents into the cache meanwhile - and, merging the context splits while it loads, the outputs.
 //   * lm_latent_attn_kernel: 16 heads of a row as the rows of one mma tile, blocks of latents through a cp.async ring and
-//     used twice, as keys and as values; eight warps share the keys for the scores and the columns for the sums.
+//     used twice, as keys and as values; the warps share the keys for the scores and the columns for the sums.
 //   * fp32 forms of both head linears; fp32 attention is that of lm_attn.cu with one head of keys.
 // Scores, weights and sums are fp32; the weights enter the second product as a sum of two bf16 numbers.
 #include <algorithm>
+#include <cmath>
+#include <type_traits>
 
 #include "../device_common.cuh"
 #include "lm_route.cuh"
@@ -151,35 +153,54 @@ __global__ void __launch_bounds__(kThreads) lm_head_linear_kernel(LatentArgs a, 
     __syncthreads();
   }
   const int k4 = K / 4, kp4 = ldx / 4;
-  for (int i = tid; i < 16 * MT * kp4; i += kThreads) {
-    const int r = i / kp4, c = i - r * kp4;
-    if (MERGE) {
-      float4 v = make_float4(0, 0, 0, 0);
-      if (r < n_here && c < k4) {
-        const float4* po = reinterpret_cast<const float4*>(a.part_o + ((size_t)(row0 + r) * a.heads + h) * splits * K) + c;
-        const float* f = sw + r * splits;
-        for (int b = 0; b < splits; b += 8) {  // eight partial rows requested together; those that do not exist weigh 0
-          float4 p[8];
+  if (MERGE) {
+    // ITEMS groups of four columns at a time, AT splits of each requested together; splits that do not exist weigh 0
+    auto merge = [&](auto items, auto at) {
+      constexpr int ITEMS = decltype(items)::value, AT = decltype(at)::value;
+      for (int i0 = tid; i0 < 16 * MT * kp4; i0 += kThreads * ITEMS) {
+        float4 v[ITEMS];
 #pragma unroll
-          for (int u = 0; u < 8; ++u) {
-            const bool in = b + u < splits && f[min(b + u, splits - 1)] != 0.0f;
-            p[u] = in ? po[(size_t)(b + u) * k4] : make_float4(0, 0, 0, 0);
+        for (int j = 0; j < ITEMS; ++j) v[j] = make_float4(0, 0, 0, 0);
+        for (int b = 0; b < splits; b += AT) {
+          float4 p[ITEMS][AT];
+          float g[ITEMS][AT];
+#pragma unroll
+          for (int j = 0; j < ITEMS; ++j) {
+            const int i = i0 + j * kThreads, r = i / kp4, c = i - r * kp4;
+            const bool ok = r < n_here && c < k4;
+            const float4* po = reinterpret_cast<const float4*>(a.part_o + ((size_t)(row0 + (ok ? r : 0)) * a.heads + h) * splits * K) + (ok ? c : 0);
+#pragma unroll
+            for (int u = 0; u < AT; ++u) {
+              g[j][u] = ok && b + u < splits ? sw[r * splits + b + u] : 0.0f;
+              p[j][u] = g[j][u] != 0.0f ? po[(size_t)(b + u) * k4] : make_float4(0, 0, 0, 0);
+            }
           }
 #pragma unroll
-          for (int u = 0; u < 8; ++u) {
-            const float g = b + u < splits ? f[b + u] : 0.0f;
-            v.x = fmaf(g, p[u].x, v.x), v.y = fmaf(g, p[u].y, v.y), v.z = fmaf(g, p[u].z, v.z), v.w = fmaf(g, p[u].w, v.w);
-          }
+          for (int j = 0; j < ITEMS; ++j)
+#pragma unroll
+            for (int u = 0; u < AT; ++u) {
+              v[j].x = fmaf(g[j][u], p[j][u].x, v[j].x), v[j].y = fmaf(g[j][u], p[j][u].y, v[j].y);
+              v[j].z = fmaf(g[j][u], p[j][u].z, v[j].z), v[j].w = fmaf(g[j][u], p[j][u].w, v[j].w);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < ITEMS; ++j) {
+          const int i = i0 + j * kThreads;
+          if (i < 16 * MT * kp4) store4(sx + i * 4, v[j]);
         }
       }
-      store4(sx + r * ldx + c * 4, v);
-    } else {
+    };
+    if constexpr (KS > 1) merge(std::integral_constant<int, 1>{}, std::integral_constant<int, 8>{});
+    else merge(std::integral_constant<int, 4>{}, std::integral_constant<int, 2>{});
+  } else {
+    for (int i = tid; i < 16 * MT * kp4; i += kThreads) {
+      const int r = i / kp4, c = i - r * kp4;
       uint2 v = make_uint2(0, 0);
       if (r < n_here && c < k4) {
         const int row = a.rows ? a.rows[row0 + r] : row0 + r;
         v = *reinterpret_cast<const uint2*>(static_cast<const __nv_bfloat16*>(a.q) + (size_t)row * a.ldq + (size_t)h * K + c * 4);
       }
-      *reinterpret_cast<uint2*>(sx + r * ldx + c * 4) = v;
+      *reinterpret_cast<uint2*>(sx + i * 4) = v;
     }
   }
   __syncthreads();
@@ -251,27 +272,40 @@ __global__ void __launch_bounds__(kThreads) lm_head_linear_f32_kernel(const floa
 }
 
 // ------------------------------------------------------------------------------------------ attention through the latent
-constexpr int kHeadRows = 16, kStages = 2;
+constexpr int kHeadRows = 16, kAttnSmemMax = 226 * 1024;
 
-int block_keys(int rankp) { return rankp <= 512 ? 64 : 32; }
-size_t attn_smem(int rankp) {
-  const int kb = block_keys(rankp);
-  return (size_t)(kHeadRows + kStages * kb) * (rankp + 8) * 2 + (size_t)kHeadRows * (kb + 4) * 4 + (size_t)2 * kHeadRows * (kb + 8) * 2;
-}
+// Shape of a CTA.  NT: tiles of 16 columns per warp; KB: keys per block; ST: blocks in the ring; NW: warps.  Scores: a warp
+// takes 8 keys and one of KQ shares of the columns, whose queries it keeps in registers if they fit (HOLD).
+template <int NT_, int KB_, int ST_, int NW_, int CTAS_>
+struct AttnCta {
+  static constexpr int NT = NT_, KB = KB_, ST = ST_, NW = NW_, CTAS = CTAS_;
+  static constexpr int kColumns = NT * NW * 16;
+  static constexpr int KQ = NW / (KB / 8);
+  static constexpr int kSteps = kColumns / 64 / KQ;  // of 64 columns, per warp
+  static constexpr bool HOLD = kSteps <= (NW * CTAS <= 8 ? 8 : 4);
+  static constexpr int LPR = 2 * NW;                 // lanes that share a row of scores
+  static constexpr int kPer = KB / LPR;
+  static constexpr int kLdS = KB + 4, kLdP = KB + 8;
+  static constexpr size_t smem(int rankp) {
+    return (size_t)(kHeadRows + ST * KB) * (rankp + 8) * 2 + (size_t)KQ * kHeadRows * kLdS * 4 + (size_t)2 * kHeadRows * kLdP * 2;
+  }
+};
+using Attn256 = AttnCta<2, 64, 2, 8, 2>;  // two CTAs of eight warps per SM: one computes while the other waits
+using Attn512 = AttnCta<4, 64, 3, 8, 1>;
+using Attn1024 = AttnCta<4, 32, 2, 16, 1>;
 
 // grid (splits, blocks of 16 heads, rows).  Leaves {max, sum} (base 2) and the unnormalized sum per split.
-// NT: tiles of 16 columns per warp; KB: keys per block, 8 per warp that computes scores.
-template <int NT, int KB>
-__global__ void __launch_bounds__(kThreads) lm_latent_attn_kernel(LatentArgs a, int chunk) {
+template <class S>
+__global__ void __launch_bounds__(S::NW * 32, S::CTAS) lm_latent_attn_kernel(LatentArgs a, int chunk) {
   extern __shared__ __align__(16) uint8_t la_smem[];
   __shared__ float s_alpha[kHeadRows];
+  constexpr int NT = S::NT, KB = S::KB, ST = S::ST, NW = S::NW, KQ = S::KQ, kLdS = S::kLdS, kLdP = S::kLdP;
   const int R = a.rankp, ldc = R + 8, splits = gridDim.x, split = blockIdx.x, idx = blockIdx.z, h0 = blockIdx.y * kHeadRows;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  constexpr int kLdS = KB + 4, kLdP = KB + 8;
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(la_smem);
   __nv_bfloat16* sC = sQ + kHeadRows * ldc;
-  __nv_bfloat16* sP = sC + kStages * KB * ldc;  // high parts, then low parts
-  float* sS = reinterpret_cast<float*>(sP + 2 * kHeadRows * kLdP);
+  __nv_bfloat16* sP = sC + ST * KB * ldc;  // high parts, then low parts
+  float* sS = reinterpret_cast<float*>(sP + 2 * kHeadRows * kLdP);  // [KQ][rows]
   pdl_launch_dependents();
   pdl_wait_prior();
   const int row = a.rows ? a.rows[idx] : idx;
@@ -282,86 +316,114 @@ __global__ void __launch_bounds__(kThreads) lm_latent_attn_kernel(LatentArgs a, 
   const __nv_bfloat16* cb = static_cast<const __nv_bfloat16*>(a.cache) + ((size_t)sp.x * a.max_ctx + j0) * R;
   const int cr = tid >> 3, cc = (tid & 7) * 8;  // copies: eight threads per row, 128 bytes at a time
   auto fetch = [&](int b) {
-    __nv_bfloat16* to = sC + (b % kStages) * KB * ldc;
+    if (b < blocks) {
+      __nv_bfloat16* to = sC + (b % ST) * KB * ldc;
+      for (int r = cr; r < KB; r += NW * 4) {
+        const int j = b * KB + r;
+        const __nv_bfloat16* src = cb + (size_t)(j < nk ? j : 0) * R + cc;
+        const uint32_t dst = smem_u32(to + r * ldc + cc);
 #pragma unroll
-    for (int u = 0; u < KB / 32; ++u) {
-      const int r = cr + u * 32, j = b * KB + r;
-      const __nv_bfloat16* src = cb + (size_t)(j < nk ? j : 0) * R;
-      for (int c = cc; c < R; c += 64) cp_async16(smem_u32(to + r * ldc + c), src + c, j < nk);
+        for (int c = 0; c < S::kColumns; c += 64)
+          if (c < R) cp_async16(dst + c * 2, src + c, j < nk);
+      }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    asm volatile("cp.async.commit_group;" ::: "memory");  // past the last block: an empty group
   };
   if (cr < kHeadRows) {
     const __nv_bfloat16* src = static_cast<const __nv_bfloat16*>(a.qa) + ((size_t)idx * a.heads + h0 + (cr < nh ? cr : 0)) * R;
     for (int c = cc; c < R; c += 64) cp_async16(smem_u32(sQ + cr * ldc + c), src + c, cr < nh);
   }
-  fetch(0);
-  const int mat = lane >> 3, ml = lane & 7;
+#pragma unroll
+  for (int b = 0; b < ST - 1; ++b) fetch(b);
+  const int mat = lane >> 3, ml = lane & 7, part = warp / (KB / 8), key = (warp % (KB / 8)) * 8;
   const uint32_t q_addr = smem_u32(sQ + ((mat & 1) * 8 + ml) * ldc + (mat >> 1) * 8);
-  const uint32_t k_addr = smem_u32(sC + (warp * 8 + ml) * ldc + mat * 8);
+  const uint32_t k_addr = smem_u32(sC + (key + ml) * ldc + mat * 8);
   const uint32_t v_addr = smem_u32(sC + ((mat & 1) * 8 + ml) * ldc + warp * NT * 16 + (mat >> 1) * 8);
   const uint32_t p_addr = smem_u32(sP + ((mat & 1) * 8 + ml) * kLdP + (mat >> 1) * 8);
   const float sc2 = a.scale * kLog2e;
-  const int srow = warp * 2 + (lane >> 4), scol = (lane & 15) * (KB / 16);  // this half-warp's row of scores
+  const int srow = tid / S::LPR, scol = (tid % S::LPR) * S::kPer;  // this lane's scores
+  uint32_t qf[S::HOLD ? 4 * S::kSteps : 4][4];
+  auto load_q = [&](uint32_t(&q)[4], int c) { ldsm4(q, q_addr + c * 2); };
+  if (S::HOLD) {
+    asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");  // the first group
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 4 * S::kSteps; ++k) {
+      const int c = ((k / 4) * KQ + part) * 64 + (k % 4) * 16;
+      qf[k][0] = qf[k][1] = qf[k][2] = qf[k][3] = 0;
+      if (c < R) load_q(qf[k], c);
+    }
+  }
   float m = kFloor, l = 0.0f, o[2 * NT][4];
 #pragma unroll
   for (int n = 0; n < 2 * NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.0f;
 
   for (int b = 0; b < blocks; ++b) {
-    const int stage = (b % kStages) * KB * ldc * 2;  // bytes
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    const int stage = (b % ST) * KB * ldc * 2;  // bytes
+    asm volatile("cp.async.wait_group %0;" ::"n"(ST - 2) : "memory");
     __syncthreads();  // the block has landed; everyone is through with the one before
-    if (b + 1 < blocks) fetch(b + 1);
-    if (warp < KB / 8) {
-      float s0[4] = {}, s1[4] = {};
-#pragma unroll 4
-      for (int k = 0; k < R; k += 32) {
-        uint32_t qa[4], qb[4], kf[4];
-        ldsm4(qa, q_addr + k * 2);
-        ldsm4(qb, q_addr + k * 2 + 32);
-        ldsm4(kf, k_addr + stage + k * 2);
-        mma_bf16(s0, qa[0], qa[1], qa[2], qa[3], kf[0], kf[1]);
-        mma_bf16(s1, qb[0], qb[1], qb[2], qb[3], kf[2], kf[3]);
+    fetch(b + ST - 1);
+    {
+      float acc[4][4] = {};
+#pragma unroll
+      for (int k = 0; k < S::kSteps; ++k) {
+        const int c = (k * KQ + part) * 64;
+        if (c < R) {
+          uint32_t kf[4], kg[4];
+          ldsm4(kf, k_addr + stage + c * 2);
+          ldsm4(kg, k_addr + stage + c * 2 + 64);
+          if (!S::HOLD)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) load_q(qf[i], c + i * 16);
+          const int q = S::HOLD ? 4 * k : 0;
+          mma_bf16(acc[0], qf[q][0], qf[q][1], qf[q][2], qf[q][3], kf[0], kf[1]);
+          mma_bf16(acc[1], qf[q + 1][0], qf[q + 1][1], qf[q + 1][2], qf[q + 1][3], kf[2], kf[3]);
+          mma_bf16(acc[2], qf[q + 2][0], qf[q + 2][1], qf[q + 2][2], qf[q + 2][3], kg[0], kg[1]);
+          mma_bf16(acc[3], qf[q + 3][0], qf[q + 3][1], qf[q + 3][2], qf[q + 3][3], kg[2], kg[3]);
+        }
       }
-      const int c = warp * 8 + (lane & 3) * 2;
-      const bool ok0 = b * KB + c < nk, ok1 = b * KB + c + 1 < nk;
-      float* st = sS + (lane >> 2) * kLdS + c;
-      *reinterpret_cast<float2*>(st) = make_float2(ok0 ? (s0[0] + s1[0]) * sc2 : kFloor, ok1 ? (s0[1] + s1[1]) * sc2 : kFloor);
-      *reinterpret_cast<float2*>(st + 8 * kLdS) = make_float2(ok0 ? (s0[2] + s1[2]) * sc2 : kFloor, ok1 ? (s0[3] + s1[3]) * sc2 : kFloor);
+      float* st = sS + (part * kHeadRows + (lane >> 2)) * kLdS + key + (lane & 3) * 2;
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[0][i] += acc[1][i] + (acc[2][i] + acc[3][i]);
+      *reinterpret_cast<float2*>(st) = make_float2(acc[0][0], acc[0][1]);
+      *reinterpret_cast<float2*>(st + 8 * kLdS) = make_float2(acc[0][2], acc[0][3]);
     }
     __syncthreads();
     {
-      float p[KB / 16], mx = m, sum = 0.0f;
+      float p[S::kPer], mx = m, sum = 0.0f;
 #pragma unroll
-      for (int i = 0; i < KB / 16; ++i) {
-        p[i] = sS[srow * kLdS + scol + i];
+      for (int i = 0; i < S::kPer; ++i) {
+        p[i] = 0.0f;
+#pragma unroll
+        for (int q = 0; q < KQ; ++q) p[i] += sS[(q * kHeadRows + srow) * kLdS + scol + i];
+        p[i] = b * KB + scol + i < nk ? p[i] * sc2 : kFloor;
         mx = fmaxf(mx, p[i]);
       }
 #pragma unroll
-      for (int d = 8; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+      for (int d = S::LPR / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
 #pragma unroll
-      for (int i = 0; i < KB / 16; ++i) {
+      for (int i = 0; i < S::kPer; ++i) {
         p[i] = fast_exp2(p[i] - mx);  // the block has a key: places without one are far below the maximum
         sum += p[i];
       }
-#pragma unroll
-      for (int d = 8; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
       const float alpha = fast_exp2(m - mx);
-      l = fmaf(l, alpha, sum);
       m = mx;
-      if ((lane & 15) == 0) s_alpha[srow] = alpha;
+      if (tid % S::LPR == 0) s_alpha[srow] = alpha;
+      __nv_bfloat16* ph = sP + srow * kLdP + scol;
 #pragma unroll
-      for (int i = 0; i < KB / 16; i += 2) {
-        const uint32_t hi = pack2(p[i], p[i + 1]);
-        const uint32_t lo = pack2(p[i] - __uint_as_float(hi << 16), p[i + 1] - __uint_as_float(hi & 0xffff0000u));
-        *reinterpret_cast<uint32_t*>(sP + srow * kLdP + scol + i) = hi;
-        *reinterpret_cast<uint32_t*>(sP + (kHeadRows + srow) * kLdP + scol + i) = lo;
+      for (int i = 0; i < S::kPer; ++i) {
+        const __nv_bfloat16 hi = __float2bfloat16_rn(p[i]);
+        ph[i] = hi;
+        ph[kHeadRows * kLdP + i] = __float2bfloat16_rn(p[i] - __bfloat162float(hi));
       }
+      l = fmaf(l, alpha, sum);  // of this lane's keys
     }
     __syncthreads();
     const float f0 = s_alpha[lane >> 2], f1 = s_alpha[(lane >> 2) + 8];
+    if (__any_sync(0xffffffffu, f0 != 1.0f || f1 != 1.0f)) {  // a new maximum: seldom after the first blocks
 #pragma unroll
-    for (int n = 0; n < 2 * NT; ++n) o[n][0] *= f0, o[n][1] *= f0, o[n][2] *= f1, o[n][3] *= f1;
+      for (int n = 0; n < 2 * NT; ++n) o[n][0] *= f0, o[n][1] *= f0, o[n][2] *= f1, o[n][3] *= f1;
+    }
 #pragma unroll
     for (int kk = 0; kk < KB / 16; ++kk) {
       uint32_t hi[4], lo[4];
@@ -380,7 +442,9 @@ __global__ void __launch_bounds__(kThreads) lm_latent_attn_kernel(LatentArgs a, 
       }
     }
   }
-  if ((lane & 15) == 0 && srow < nh) a.part_ml[((size_t)idx * a.heads + h0 + srow) * splits + split] = make_float2(m, l);
+#pragma unroll
+  for (int d = S::LPR / 2; d > 0; d >>= 1) l += __shfl_xor_sync(0xffffffffu, l, d);
+  if (tid % S::LPR == 0 && srow < nh) a.part_ml[((size_t)idx * a.heads + h0 + srow) * splits + split] = make_float2(m, l);
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int r = (lane >> 2) + i * 8;
@@ -393,17 +457,16 @@ __global__ void __launch_bounds__(kThreads) lm_latent_attn_kernel(LatentArgs a, 
 }
 
 // ------------------------------------------------------------------------------------------ launches
-constexpr int kMaxCtxSplits = 128;
-
 struct Split {
   int chunk, splits;
 };
-// Context per CTA: as many CTAs as fit the GPU at once, if there are that many blocks of keys.
+// Context per CTA: as many CTAs as fit the GPU at once, but no more splits than pay: a block more in a row costs about four
+// times what a split more costs the merge.
 Split split_context(const LatentArgs& a) {
-  const int kb = block_keys(a.rankp), hblocks = (a.heads + kHeadRows - 1) / kHeadRows;
-  const int fit = std::max(1, std::min(3, (int)(220 * 1024 / (attn_smem(a.rankp) + 1024))));
-  const int want = std::max(1, std::min(kMaxCtxSplits, kSms * fit / (a.n_rows * hblocks)));
-  const int blocks = (a.ctx + kb - 1) / kb, per = (blocks + want - 1) / want;
+  const int kb = a.rankp <= 512 ? Attn512::KB : Attn1024::KB, fit = a.rankp <= 256 ? Attn256::CTAS : 1;
+  const int blocks = (a.ctx + kb - 1) / kb, hblocks = (a.heads + kHeadRows - 1) / kHeadRows;
+  const int want = std::max(1, std::min((int)std::ceil(2.0 * std::sqrt((double)blocks)), kSms * fit / (a.n_rows * hblocks)));
+  const int per = (blocks + want - 1) / want;
   return {per * kb, (blocks + per - 1) / per};
 }
 
@@ -411,36 +474,36 @@ size_t head_linear_smem(int mt, int K, int splits) { return (size_t)16 * mt * ((
 
 template <bool MERGE>
 cudaError_t launch_head_linear(cudaStream_t s, const LatentArgs& a, int N, int K, Split sp, bool cache_rows) {
-  const int mt = a.n_rows <= 16 ? 1 : a.n_rows <= 32 ? 2 : 4;
+  const int mt = MERGE || a.n_rows <= 16 ? 1 : a.n_rows <= 32 ? 2 : 4;  // merging is the longer part: more CTAs
   const bool fine = MERGE && a.n_rows <= 8 && K >= 128;  // few rows: more CTAs, K shared by four warps
   const int cols = fine ? 16 : 64, slices = (N + cols - 1) / cols;
   const dim3 grid(a.heads * slices + (cache_rows ? 16 * mt / kWarps : 0), (a.n_rows + 16 * mt - 1) / (16 * mt));
   const size_t smem = head_linear_smem(mt, K, MERGE ? sp.splits : 0);
   auto go = [&](auto f) { return launch_pdl(f, grid, dim3(kThreads), smem, s, a, N, K, slices, sp.chunk, sp.splits); };
-  if (fine) return go(lm_head_linear_kernel<1, 4, MERGE>);
-  return mt == 1 ? go(lm_head_linear_kernel<1, 1, MERGE>) : mt == 2 ? go(lm_head_linear_kernel<2, 1, MERGE>) : go(lm_head_linear_kernel<4, 1, MERGE>);
+  if constexpr (MERGE) {
+    return fine ? go(lm_head_linear_kernel<1, 4, true>) : go(lm_head_linear_kernel<1, 1, true>);
+  } else {
+    return mt == 1 ? go(lm_head_linear_kernel<1, 1, false>) : mt == 2 ? go(lm_head_linear_kernel<2, 1, false>) : go(lm_head_linear_kernel<4, 1, false>);
+  }
 }
 
 }  // namespace
 
-size_t latent_parts(int rows) { return std::max((size_t)rows, (size_t)3 * kSms); }
+size_t latent_parts(int rows) { return std::max((size_t)rows, (size_t)2 * kSms); }
 
 cudaError_t latent_configure() {
   cudaError_t r = cudaSuccess;
-  auto set = [&](auto f) {
-    if (r == cudaSuccess) r = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024);
+  auto set = [&](auto f, int most = 200 * 1024) {
+    if (r == cudaSuccess) r = cudaFuncSetAttribute(f, cudaFuncAttributeMaxDynamicSharedMemorySize, most);
   };
-  set(lm_latent_attn_kernel<1, 64>);
-  set(lm_latent_attn_kernel<2, 64>);
-  set(lm_latent_attn_kernel<4, 64>);
-  set(lm_latent_attn_kernel<8, 32>);
+  set(lm_latent_attn_kernel<Attn256>, kAttnSmemMax);
+  set(lm_latent_attn_kernel<Attn512>, kAttnSmemMax);
+  set(lm_latent_attn_kernel<Attn1024>, kAttnSmemMax);
   set(lm_head_linear_kernel<1, 1, false>);
   set(lm_head_linear_kernel<2, 1, false>);
   set(lm_head_linear_kernel<4, 1, false>);
   set(lm_head_linear_kernel<1, 4, true>);
   set(lm_head_linear_kernel<1, 1, true>);
-  set(lm_head_linear_kernel<2, 1, true>);
-  set(lm_head_linear_kernel<4, 1, true>);
   return r;
 }
 
@@ -475,11 +538,11 @@ cudaError_t launch_latent_absorbed(cudaStream_t s, bool f32, const LatentArgs& a
   cudaError_t r = launch_head_linear<false>(s, a, a.rankp, a.dimp, sp, cache_rows);
   if (r != cudaSuccess) return r;
   const dim3 grid(sp.splits, (a.heads + kHeadRows - 1) / kHeadRows, a.n_rows);
-  auto go = [&](auto f) { return launch_pdl(f, grid, dim3(kThreads), attn_smem(a.rankp), s, a, sp.chunk); };
-  r = a.rankp <= 128   ? go(lm_latent_attn_kernel<1, 64>)
-      : a.rankp <= 256 ? go(lm_latent_attn_kernel<2, 64>)
-      : a.rankp <= 512 ? go(lm_latent_attn_kernel<4, 64>)
-                       : go(lm_latent_attn_kernel<8, 32>);
+  auto go = [&](auto shape) {
+    using S = decltype(shape);
+    return launch_pdl(lm_latent_attn_kernel<S>, grid, dim3(S::NW * 32), S::smem(a.rankp), s, a, sp.chunk);
+  };
+  r = a.rankp <= 256 ? go(Attn256{}) : a.rankp <= 512 ? go(Attn512{}) : go(Attn1024{});
   if (r != cudaSuccess) return r;
   return launch_head_linear<true>(s, a, a.vdimp, a.rankp, sp, false);
 }

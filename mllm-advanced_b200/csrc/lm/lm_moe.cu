@@ -21,9 +21,12 @@ __global__ void __launch_bounds__(kTopkWarps * 32) lm_topk_kernel(RouterArgs a, 
   float* z = z_all + (size_t)warp * a.experts;
   const float* src = logits + (size_t)row * ldl;
   for (int e = lane; e < a.experts; e += 32) {
-    float v = src[e];
-    for (int p = 1; p < planes; ++p) v += src[p * plane + e];
-    z[e] = v + a.b[e];
+    float p[kMaxSplits], v = a.b[e];
+#pragma unroll
+    for (int i = 0; i < kMaxSplits; ++i) p[i] = i < planes ? src[i * plane + e] : 0.0f;
+#pragma unroll
+    for (int i = 0; i < kMaxSplits; ++i) v += p[i];
+    z[e] = v;
   }
   __syncwarp();
   choose_experts(z, a, row, lane);

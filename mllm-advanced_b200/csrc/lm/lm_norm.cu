@@ -1,5 +1,7 @@
 // Row operators of the language-model engine: embedding, sandwich norm with residual and causal input convolution, norm
 // behind the residual sum (with the choice of experts), the bookkeeping of a decode step, and the argmax candidates of greedy sampling.
+#include <cooperative_groups.h>
+
 #include <algorithm>
 
 #include "../device_common.cuh"
@@ -319,13 +321,18 @@ cudaError_t launch_norm_t(cudaStream_t s, const NormArgs& a) {
   return cudaErrorInvalidValue;
 }
 
-// x' = rms_unit(alpha x + delta) * gain, a CTA per row; with a router the CTA goes on to choose the row's experts.
-template <class T, int NV>
+// x' = rms_unit(alpha x + delta) * gain, a CTA per row.  With a router a cluster of CTAs per row: each makes the row and
+// the logits of its share of the experts, the first one keeps the row and chooses.
+template <class T, int NV, bool ROUTER>
 __global__ void __launch_bounds__(kNormThreads) lm_post_norm_kernel(PostNormArgs a) {
   extern __shared__ __align__(16) float row_x[];  // [ldx], then [experts]; with a router only
   __shared__ float scratch[32];
-  const int tid = threadIdx.x, nv = a.ldx >> 2, t = blockIdx.x;
+  const int tid = threadIdx.x, nv = a.ldx >> 2, t = blockIdx.x, part = ROUTER ? blockIdx.y : 0, parts = ROUTER ? gridDim.y : 1;
   pdl_launch_dependents();
+  if (ROUTER)  // the router's weights do not depend on the previous kernel: into L2, a share per row and CTA
+    for (size_t at = ((size_t)(t * parts + part) * kNormThreads + tid) * 64, step = (size_t)gridDim.x * parts * kNormThreads * 64;
+         at < (size_t)a.router.experts * a.router.ldw; at += step)
+      asm volatile("prefetch.global.L2 [%0];" ::"l"(a.router.w + at));
   float4 g[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
@@ -347,43 +354,53 @@ __global__ void __launch_bounds__(kNormThreads) lm_post_norm_kernel(PostNormArgs
     ss += dot4(x[i]);
   }
   const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)a.width + a.eps);
+  auto keep_row = [&]() {
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = tid + i * kNormThreads;
+      if (c >= nv) continue;
+      if (a.x_out) store4(a.x_out + (size_t)t * a.ldx + c * 4, x[i]);
+      store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c * 4, x[i]);
+    }
+  };
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
+    x[i] = make_float4(x[i].x * r * g[i].x, x[i].y * r * g[i].y, x[i].z * r * g[i].z, x[i].w * r * g[i].w);
     const int c = tid + i * kNormThreads;
-    if (c >= nv) continue;
-    const float4 y = make_float4(x[i].x * r * g[i].x, x[i].y * r * g[i].y, x[i].z * r * g[i].z, x[i].w * r * g[i].w);
-    if (a.x_out) store4(a.x_out + (size_t)t * a.ldx + c * 4, y);
-    store4(static_cast<T*>(a.out) + (size_t)t * a.ldx + c * 4, y);
-    if (a.router.w) store4(row_x + c * 4, y);
+    if (ROUTER && c < nv) store4(row_x + c * 4, x[i]);
   }
-  if (!a.router.w) return;
+  if (!ROUTER) {
+    keep_row();
+    return;
+  }
   __syncthreads();
-  float* z = row_x + a.ldx;
-  const int warp = tid >> 5, lane = tid & 31;
-  for (int e0 = warp; e0 < a.router.experts; e0 += kNormThreads / 16) {  // two experts at a time
-    const int e1 = e0 + kNormThreads / 32;
-    const bool two = e1 < a.router.experts;
-    const __nv_bfloat16 *w0 = a.router.w + (size_t)e0 * a.router.ldw, *w1 = two ? w0 + (size_t)(kNormThreads / 32) * a.router.ldw : w0;
-    float s0 = 0.0f, s1 = 0.0f;
+  auto cluster = cooperative_groups::this_cluster();
+  float* z = cluster.map_shared_rank(row_x + a.ldx, 0);  // the logits meet in the first CTA
+  const int warp = tid >> 5, lane = tid & 31, step = parts * (kNormThreads / 32);
+  constexpr int kAtOnce = 4;
+  for (int e0 = part * (kNormThreads / 32) + warp; e0 < a.router.experts; e0 += step * kAtOnce) {
+    float s[kAtOnce] = {};
 #pragma unroll 4
     for (int c = lane * 8; c < a.ldx; c += 256) {
-      const uint4 p = __ldg(reinterpret_cast<const uint4*>(w0 + c)), q = __ldg(reinterpret_cast<const uint4*>(w1 + c));
       const float4 u = *reinterpret_cast<const float4*>(row_x + c), v = *reinterpret_cast<const float4*>(row_x + c + 4);
-      s0 += dot8(p, u, v);
-      s1 += dot8(q, u, v);
+#pragma unroll
+      for (int j = 0; j < kAtOnce; ++j) {
+        const int e = min(e0 + j * step, a.router.experts - 1);
+        s[j] += dot8(__ldg(reinterpret_cast<const uint4*>(a.router.w + (size_t)e * a.router.ldw + c)), u, v);
+      }
     }
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      s0 += __shfl_xor_sync(0xffffffffu, s0, o);
-      s1 += __shfl_xor_sync(0xffffffffu, s1, o);
-    }
-    if (lane == 0) {
-      z[e0] = s0 + a.router.b[e0];
-      if (two) z[e1] = s1 + a.router.b[e1];
+    for (int j = 0; j < kAtOnce; ++j) {
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) s[j] += __shfl_xor_sync(0xffffffffu, s[j], o);
+      const int e = e0 + j * step;
+      if (lane == 0 && e < a.router.experts) z[e] = s[j] + a.router.b[e];
     }
   }
-  __syncthreads();
-  if (warp == 0) choose_experts(z, a.router, t, lane);
+  cluster.sync();  // also: every CTA has read the row, which x_out may overwrite
+  if (part) return;
+  keep_row();
+  if (warp == 0) choose_experts(row_x + a.ldx, a.router, t, lane);
 }
 
 // The same for many rows, a warp per row.
@@ -426,12 +443,15 @@ constexpr int kFusedRouterRows = 2 * kSms;
 
 template <class T, int NV>
 cudaError_t launch_post_norm_nv(cudaStream_t s, const PostNormArgs& a) {
-  const size_t smem = a.router.w ? (size_t)(a.ldx + a.router.experts) * sizeof(float) : 0;
-  return launch_pdl(lm_post_norm_kernel<T, NV>, dim3(a.rows), dim3(kNormThreads), smem, s, a);
+  if (!a.router.w) return launch_pdl(lm_post_norm_kernel<T, NV, false>, dim3(a.rows), dim3(kNormThreads), 0, s, a);
+  int parts = 8;
+  while (parts > 1 && (a.rows * parts > 2 * kSms || a.router.experts < parts * (kNormThreads / 32))) parts /= 2;
+  const size_t smem = (size_t)(a.ldx + a.router.experts) * sizeof(float);
+  return launch_pdl_cluster(lm_post_norm_kernel<T, NV, true>, dim3(a.rows, parts), dim3(kNormThreads), dim3(1, parts, 1), smem, s, a);
 }
 template <class T>
 cudaError_t launch_post_norm_t(cudaStream_t s, const PostNormArgs& a) {
-  if (a.rows > kFusedRouterRows && !a.gather && !a.router.w && a.ldx <= 4096) {
+  if (a.rows > 16 * kSms && !a.gather && !a.router.w && a.ldx <= 4096) {
     const int w = (a.ldx / 4 + 31) / 32;
     const dim3 grid((a.rows + kNormThreads / 32 - 1) / (kNormThreads / 32));
     if (w <= 8) return launch_pdl(lm_post_norm_rows_kernel<T, 8>, grid, dim3(kNormThreads), 0, s, a);

@@ -23,11 +23,19 @@ __device__ __forceinline__ void choose_experts(float* z, const RouterArgs& a, in
   constexpr float kUsed = -3.402823466e+38f;
   float mine = 0.0f, first = 0.0f;
   int mine_e = 0;
-  for (int k = 0; k < a.top; ++k) {
-    float bv = kUsed;
-    int be = 0x7fffffff;
+  // a lane's own candidate is looked for again only after it was chosen
+  float own = kUsed;
+  int own_e = 0x7fffffff;
+  auto look = [&]() {
+    own = kUsed;
+    own_e = 0x7fffffff;
     for (int e = lane; e < a.experts; e += 32)
-      if (z[e] > bv) bv = z[e], be = e;
+      if (z[e] > own) own = z[e], own_e = e;
+  };
+  look();
+  for (int k = 0; k < a.top; ++k) {
+    float bv = own;
+    int be = own_e;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) {
       const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
@@ -37,8 +45,10 @@ __device__ __forceinline__ void choose_experts(float* z, const RouterArgs& a, in
     be = min(be, a.experts - 1);  // logits that are not numbers
     if (k == 0) first = bv;
     if (lane == k) mine = bv, mine_e = be;
-    if (lane == 0) z[be] = kUsed;
-    __syncwarp();
+    if (be == own_e) {
+      z[be] = kUsed;
+      look();
+    }
   }
   const float p = lane < a.top ? expf(mine - first) : 0.0f;
   float sum = p;

@@ -431,7 +431,8 @@ def needle_model(heads, dim, vdim, rank, shared=False, score=12.0):
 
 @gpu
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,dim,vdim,rank,shared", [(4, 32, 24, 48, False), (17, 16, 16, 200, False), (2, 64, 40, 72, True), (1, 16, 16, 640, False)])
+@pytest.mark.parametrize("heads,dim,vdim,rank,shared", [(4, 32, 24, 48, False), (17, 16, 16, 200, False), (2, 64, 40, 72, True), (3, 16, 16, 256, False),
+                                                         (3, 16, 16, 512, False), (1, 16, 16, 640, False), (2, 16, 16, 1024, False)])
 def test_one_far_key_at_every_distance(dtype, heads, dim, vdim, rank, shared, tmp_path):
     """NEEDLE at distances around key blocks, row tiles and context splits; ASK in a prompt, in a short portion, and
     decoded; a second NEEDLE right behind ASK must not be seen."""
