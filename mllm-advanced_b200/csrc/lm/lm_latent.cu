@@ -161,7 +161,8 @@ __global__ void __launch_bounds__(kThreads) lm_head_linear_kernel(LatentArgs a, 
         float4 v[ITEMS];
 #pragma unroll
         for (int j = 0; j < ITEMS; ++j) v[j] = make_float4(0, 0, 0, 0);
-        for (int b = 0; b < splits; b += AT) {
+        const int last = n_here * kp4;  // later places are padding rows
+        for (int b = 0; b < splits && i0 < last; b += AT) {
           float4 p[ITEMS][AT];
           float g[ITEMS][AT];
 #pragma unroll
@@ -291,7 +292,7 @@ struct AttnCta {
   }
 };
 using Attn256 = AttnCta<2, 64, 2, 8, 2>;  // two CTAs of eight warps per SM: one computes while the other waits
-using Attn512 = AttnCta<4, 64, 3, 8, 1>;
+using Attn512 = AttnCta<4, 64, 2, 8, 1>;
 using Attn1024 = AttnCta<4, 32, 2, 16, 1>;
 
 // grid (splits, blocks of 16 heads, rows).  Leaves {max, sum} (base 2) and the unnormalized sum per split.
@@ -460,12 +461,12 @@ __global__ void __launch_bounds__(S::NW * 32, S::CTAS) lm_latent_attn_kernel(Lat
 struct Split {
   int chunk, splits;
 };
-// Context per CTA: as many CTAs as fit the GPU at once, but no more splits than pay: a block more in a row costs about four
-// times what a split more costs the merge.
+// Context per CTA: as many CTAs as fit the GPU at once, but no more splits than pay (a split more costs the merge a
+// twenty-fifth of what a block more in a row costs).
 Split split_context(const LatentArgs& a) {
   const int kb = a.rankp <= 512 ? Attn512::KB : Attn1024::KB, fit = a.rankp <= 256 ? Attn256::CTAS : 1;
   const int blocks = (a.ctx + kb - 1) / kb, hblocks = (a.heads + kHeadRows - 1) / kHeadRows;
-  const int want = std::max(1, std::min((int)std::ceil(2.0 * std::sqrt((double)blocks)), kSms * fit / (a.n_rows * hblocks)));
+  const int want = std::max(1, std::min((int)std::ceil(5.0 * std::sqrt((double)blocks)), kSms * fit / (a.n_rows * hblocks)));
   const int per = (blocks + want - 1) / want;
   return {per * kb, (blocks + per - 1) / per};
 }
